@@ -1,11 +1,16 @@
-"""Model families assembled from the add-on layers: GPT-2, GPT-J and Llama shaped decoders, their training program
-(`DecoderTrainer`) and the int4 tensor-parallel decoding program (`DecoderGenerator`)."""
+"""Model families: GPT-2, GPT-J and Llama shaped decoders assembled from the add-on layers, their training program
+(`DecoderTrainer`) and the int4 tensor-parallel decoding program (`DecoderGenerator`); Dunelix, served from a checkpoint
+folder by `SequenceGenerator`; the registry of architectures (`load_model`)."""
 from .decoder import DecoderBlock, DecoderConfig, DecoderEmbedding, DecoderHead
 
 __all__ = ["DecoderConfig", "DecoderBlock", "DecoderEmbedding", "DecoderHead", "DecoderTrainer", "PipelineTrainer",
-           "DecoderGenerator"]
+           "DecoderGenerator", "Dunelix", "DunelixConfig", "SequenceGenerator", "load_model", "load_config",
+           "register_architecture", "ARCHITECTURES"]
 
-_LAZY = {"DecoderTrainer": "trainer", "PipelineTrainer": "pipeline_trainer", "DecoderGenerator": "generator"}
+_LAZY = {"DecoderTrainer": "trainer", "PipelineTrainer": "pipeline_trainer", "DecoderGenerator": "generator",
+         "Dunelix": "dunelix", "DunelixConfig": "dunelix", "SequenceGenerator": "sequence_generator",
+         "load_model": "registry", "load_config": "registry", "register_architecture": "registry",
+         "ARCHITECTURES": "registry"}
 
 
 def __getattr__(name):

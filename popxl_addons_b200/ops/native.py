@@ -1545,3 +1545,5 @@ def _register_late():
 
 
 _register_late()
+
+from . import native_sequence  # noqa: E402,F401  (kernels of the sequence-model ops)

@@ -1,0 +1,160 @@
+"""CUDA implementations of the sequence-model ops (`xl/ops/sequence.py`): bf16 models run hand-written kernels throughout;
+32-bit models use plain fp32 matrix products (never a reduced-precision matrix mode) and the same kernels for the rest."""
+import torch
+
+from ..xl.opdef import OPS, native
+from .native import (_CODE, _c_f, _c_int, _c_ll, _c_p, _check, _count, _ok, _sig, _stream, gemm)
+
+_stream_dyt = _sig("xl_stream_dyt", _c_p, _c_p, _c_f, _c_p, _c_p, _c_int, _c_p, _c_p, _c_p, _c_p, _c_ll, _c_int, _c_int, _c_p)
+_select_dyt = _sig("xl_select_dyt", _c_p, _c_p, _c_int, _c_int, _c_ll, _c_p, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int, _c_p)
+_swiglu_packed = _sig("xl_swiglu_packed", _c_p, _c_p, _c_ll, _c_int, _c_int, _c_p)
+_advance_by = _sig("xl_advance_by", _c_p, _c_p, _c_int, _c_p)
+_min_gru = _sig("xl_min_gru", _c_p, _c_p, _c_p, _c_p, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int, _c_p)
+_rope_append = _sig("xl_diff_rope_append", _c_p, _c_ll, _c_p, _c_p, _c_p, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int,
+                    _c_int, _c_int, _c_int, _c_int, _c_int, _c_p)
+_diff_general = _sig("xl_diff_attn_general", _c_p, _c_ll, _c_p, _c_p, _c_p, _c_ll, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int,
+                     _c_int, _c_int, _c_int, _c_int, _c_int, _c_f, _c_f, _c_f, _c_int, _c_p)
+
+
+def _ptr(t):
+    return t.data_ptr() if t is not None else None
+
+
+def _f32(*ts) -> bool:
+    return all(t is None or t.dtype == torch.float32 for t in ts)
+
+
+def _i32(*ts) -> bool:
+    return all(t is None or (t.is_cuda and t.is_contiguous() and t.dtype == torch.int32) for t in ts)
+
+
+def product(a, weight, out_dtype=None):
+    """`a (n, K) @ weight (N, K)^T` with 32-bit accumulation: the tcgen05 GEMM for 16-bit operands, the vendor product for
+    sizes it does not take and for 32-bit models."""
+    out_dtype = out_dtype or a.dtype
+    if a.dtype != torch.float32:
+        y = gemm(a, weight.t(), out_dtype=out_dtype)
+        if y is not NotImplemented:
+            return y
+        y = torch.mm(a, weight.t())
+        return y if y.dtype == out_dtype else y.to(out_dtype)
+    if torch.backends.cuda.matmul.allow_tf32:
+        raise RuntimeError("32-bit models need true fp32 matrix products: set torch.backends.cuda.matmul.allow_tf32 = False")
+    return torch.mm(a, weight.t()).to(out_dtype)
+
+
+def stream_dyt(x, y, mult, tokens, table, norm, out_dtype):
+    """One pass over the residual stream: `x += mult * y (+ table[tokens])`, or `x = table[tokens]` without `y`; returns the
+    Dynamic Tanh of it when `norm` is given."""
+    rows = y.shape[0] if y is not None else tokens.numel()
+    cols = x.shape[1]
+    if not _ok(x, y, table) or not _f32(x, *(norm or ())) or not _i32(tokens) or rows > x.shape[0]:
+        return NotImplemented
+    alpha, w, b = norm if norm is not None else (None, None, None)
+    if norm is not None and not _ok(w, b):
+        return NotImplemented
+    h = torch.empty((rows, cols), dtype=out_dtype, device=x.device) if norm is not None else None
+    rc = _stream_dyt(x.data_ptr(), _ptr(y), float(mult), _ptr(tokens), _ptr(table), table.shape[0] if table is not None else 0,
+                     _ptr(alpha), _ptr(w), _ptr(b), _ptr(h), rows, cols, _CODE[out_dtype], _stream())
+    if rc == -1:
+        return NotImplemented
+    _check(rc, "stream_dyt")
+    _count("stream_dyt")
+    return h if norm is not None else ()
+
+
+@native("embed_dyt_")
+def embed_dyt_cuda(x, tokens, table, alpha, w, b):
+    return stream_dyt(x, None, 0.0, tokens.reshape(-1), table, (alpha, w, b), table.dtype)
+
+
+@native("linear_residual_dyt_")
+def linear_residual_dyt_cuda(x, a, weight, *rest, mult, has_norm, has_inject):
+    norm = rest[:3] if has_norm else None
+    tokens, table = rest[-2:] if has_inject else (None, None)
+    y = product(a, weight)
+    return stream_dyt(x, y, mult, tokens.reshape(-1) if tokens is not None else None, table, norm, a.dtype)
+
+
+@native("select_dyt")
+def select_dyt_cuda(x, idx, alpha, w, b, stride, offset, out_dtype):
+    if not _ok(x) or not _f32(x, alpha, w, b) or not _i32(idx):
+        return NotImplemented
+    h = torch.empty((idx.shape[0], x.shape[1]), dtype=out_dtype, device=x.device)
+    rc = _select_dyt(x.data_ptr(), idx.data_ptr(), stride, offset, x.shape[0], alpha.data_ptr(), w.data_ptr(), b.data_ptr(),
+                     h.data_ptr(), idx.shape[0], x.shape[1], _CODE[out_dtype], _stream())
+    if rc == -1:
+        return NotImplemented
+    _check(rc, "select_dyt")
+    _count("select_dyt")
+    return h
+
+
+@native("linear_rows")
+def linear_rows_cuda(a, weight, out_dtype):
+    return product(a, weight, out_dtype)
+
+
+@native("linear_swiglu")
+def linear_swiglu_cuda(h, weight):
+    f = weight.shape[0] // 2
+    gu = product(h, weight)
+    y = torch.empty((h.shape[0], f), dtype=h.dtype, device=h.device)
+    rc = _swiglu_packed(gu.data_ptr(), y.data_ptr(), h.shape[0], f, _CODE[h.dtype], _stream())
+    _check(rc, "swiglu_packed")
+    _count("swiglu_packed")
+    return y
+
+
+@native("min_gru_")
+def min_gru_cuda(h, weight, bz, bx, state, pos, count, T):
+    B, width = state.shape
+    if not _f32(bz, bx, state) or not _i32(pos, count) or not state.is_contiguous() or h.shape[0] != B * T:
+        return NotImplemented
+    zxg = product(h, weight)
+    y = torch.empty((B * T, width), dtype=h.dtype, device=h.device)
+    rc = _min_gru(zxg.data_ptr(), bz.data_ptr(), bx.data_ptr(), state.data_ptr(), y.data_ptr(), pos.data_ptr(),
+                  count.data_ptr(), B, T, width, _CODE[h.dtype], _stream())
+    if rc == -1:
+        return NotImplemented
+    _check(rc, "min_gru")
+    _count("min_gru")
+    return y
+
+
+@native("diff_attention_")
+def diff_attention_cuda(qkv, cos, sin, kc, vc, pos, count, lam, T, heads, rotary_dim, chunk, scale, eps, out_scale):
+    B, G, _, smax, dim = kc.shape
+    vdim = vc.shape[-1]
+    if not _ok(qkv, kc, vc) or not (qkv.dtype == kc.dtype == vc.dtype) or not _f32(cos, sin, lam) or not _i32(pos, count):
+        return NotImplemented
+    if qkv.shape != (B * T, (heads + G) * 2 * dim + G * vdim) or (rotary_dim and cos.shape[0] < smax):
+        return NotImplemented
+    code, s = _CODE[qkv.dtype], _stream()
+    out = torch.empty((B * T, heads * vdim), dtype=qkv.dtype, device=qkv.device)
+    rc = _rope_append(qkv.data_ptr(), qkv.stride(0), _ptr(cos), _ptr(sin), kc.data_ptr(), vc.data_ptr(), pos.data_ptr(),
+                      count.data_ptr(), B, T, heads, G, dim, vdim, rotary_dim, smax, code, s)
+    if rc == -1:
+        return NotImplemented
+    _check(rc, "diff_rope_append")
+    _count("diff_rope_append")
+    rc = _diff_general(qkv.data_ptr(), qkv.stride(0), kc.data_ptr(), vc.data_ptr(), out.data_ptr(), out.stride(0),
+                       pos.data_ptr(), count.data_ptr(), lam.data_ptr(), B, T, heads, G, dim, vdim, smax, chunk, float(scale),
+                       float(eps), float(out_scale), code, s)
+    _check(rc, "diff_attn_general")
+    _count("diff_attn_general")
+    return out
+
+
+@native("advance_by_")
+def advance_by_cuda(pos, count):
+    if not _i32(pos, count):
+        return NotImplemented
+    _check(_advance_by(pos.data_ptr(), count.data_ptr(), pos.numel(), _stream()), "advance_by")
+    _count("advance_by")
+    return pos
+
+
+# kept importable by name for tests that drive one kernel at a time
+__all__ = ["product", "stream_dyt"] + [n for n in list(globals()) if n.endswith("_cuda")]
+assert "diff_attention_" in OPS

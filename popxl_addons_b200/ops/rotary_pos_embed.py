@@ -2,14 +2,14 @@
 
 Parity: popxl_addons/ops/rotary_pos_embed/rotary_pos_embed.py:19-109.
 """
-from typing import Optional, Tuple
+from typing import Mapping, Optional, Tuple
 
 import numpy as np
 
 from .. import xl
 from ..xl import ops
 
-__all__ = ["rotary_pos_embed", "trig_tables", "trig_table_constants"]
+__all__ = ["rotary_pos_embed", "trig_tables", "trig_table_constants", "rotary_frequencies", "frequency_tables"]
 
 
 def trig_tables(seq_len: int, rotary_dim: int, base: int = 10000, np_dtype="float32",
@@ -27,6 +27,26 @@ def trig_table_constants(seq_len: int, rotary_dim: int, base: int = 10000, dtype
     """`(sin, cos)` constants of shape `(seq_len, rotary_dim/2)`."""
     sin, cos = trig_tables(seq_len, rotary_dim, base)
     return xl.constant(sin, dtype, "rotary_sin"), xl.constant(cos, dtype, "rotary_cos")
+
+
+def rotary_frequencies(rotary_dim: int, base: float, scaling: Optional[Mapping[str, float]] = None) -> np.ndarray:
+    """Angle per position of every feature pair, `base^(-2i/rotary_dim)` (float64). `scaling` = `factor, low, high,
+    original` stretches the long wavelengths as Llama 3.1 does: pairs that turn more than `high` times within `original`
+    positions stay, those that turn less than `low` times are slowed by `factor`, with a linear blend in between."""
+    f = np.power(float(base), -np.arange(0, rotary_dim, 2, dtype=np.float64) / rotary_dim)
+    if not scaling:
+        return f
+    factor, low, high, original = (float(scaling[k]) for k in ("factor", "low", "high", "original"))
+    turns = original * f / (2.0 * np.pi)
+    blend = (turns - low) / (high - low) if high != low else np.zeros_like(turns)
+    mixed = (1.0 - blend) * f / factor + blend * f
+    return np.where(turns > high, f, np.where(turns < low, f / factor, mixed))
+
+
+def frequency_tables(seq_len: int, freqs: np.ndarray) -> Tuple[np.ndarray, np.ndarray]:
+    """`(sin, cos)` float32 tables `(seq_len, len(freqs))` of the angles `m * freqs`, evaluated in float64."""
+    angle = np.outer(np.arange(seq_len, dtype=np.float64), np.asarray(freqs, np.float64))
+    return np.sin(angle).astype(np.float32), np.cos(angle).astype(np.float32)
 
 
 def rotary_pos_embed(t: xl.Tensor, sin: xl.Tensor, cos: xl.Tensor, rotary_dim: Optional[int] = None) -> xl.Tensor:

@@ -14,6 +14,7 @@ from . import ops
 from . import transforms
 from .autodiff import ExpectedConnection, ExpectedConnectionType, GradGraphInfo
 from .session import Session
+from .program import Program
 from .ops.control import CallSiteInfo
 
 bool = bool_  # noqa: A001  (popxl exposes the boolean dtype under this name)

@@ -102,6 +102,7 @@ class Session:
         self._slab_events: Dict[RemoteBuffer, tuple] = {}  # last access of a remote-buffer slab: (event, stream id)
         self._slab_pending = None
         self._uncapturable: set = set()        # loops whose capture failed once: they run eagerly from then on
+        self._programs: Dict[Any, Any] = {}    # program -> captured state (None: run once, not captured yet)
         self._init_state()
 
     # ------------------------------------------------------------------------------------------------------
@@ -962,4 +963,39 @@ class Session:
             _native.check_gemm_errors()
             if getattr(self, "_fused_runtime", None) is not None:
                 self._fused_runtime.check()
+        return out
+
+    def run_program(self, program, inputs: Optional[Mapping[HostToDeviceStream, Any]] = None,
+                    fetch: bool = True) -> Dict[DeviceToHostStream, np.ndarray]:
+        """Execute a `Program` once; inputs, outputs and `fetch` as in `run`. The first run is eager (lazy
+        initialisation); a capturable program is captured into a CUDA graph at its second run and replayed from then on."""
+        self._outputs = {}
+        self._stage_inputs(inputs or {})
+        with torch.no_grad():
+            state = self._programs.get(program)
+            capturable = (program.capture and self.device.type == "cuda" and self.num_local == 1 and self.profile is None
+                          and self.ir.options.cuda_graphs)
+            if state is not None and capturable:
+                from ..ops import native as _native
+
+                for stream, static in state["static_in"].items():
+                    static.copy_(self._next_host_item(stream), non_blocking=True)
+                state["graph"].replay()
+                _native.count_replay(state["kernels"])
+                self._after_replay(state)
+            else:
+                vals = [self._value(t, {}) for t in program.bindings.values()]
+                if capturable and program in self._programs and self._capture_safe(program.graph):
+                    state = self._capture(None, program.graph, vals, [])
+                    self._programs[program] = state
+                    self._after_replay(state)
+                else:
+                    self.run_graph(program.graph, vals)
+                    self._join_streams()
+                    self._programs.setdefault(program, None)
+        out = self._collect_outputs(fetch)
+        if self.use_native and fetch:
+            from ..ops import native as _native
+
+            _native.check_gemm_errors()
         return out

@@ -12,6 +12,7 @@
 //
 //   xl_diff_rope_append    rotate q in place, k into the cache, v into the cache
 //   xl_diff_attn_general   any sizes and types, scores and weights in fp32 on the CUDA cores: one warp per row and head
+//   xl_diff_attn_decode    one token per sequence, bf16: rotation, append, attention and the combination in one launch
 #include "common.cuh"
 
 #include <math.h>
@@ -148,6 +149,348 @@ __global__ void __launch_bounds__(DG_WARPS * 32)
     if (lane + 32 * e < vdim) out[row * ldo + (long long)h * vdim + lane + 32 * e] = xl_from_float<T>(c[e] * f);
 }
 
+// ---- decoding: one query row per sequence ------------------------------------------------------------------------------
+// Grid (splits, G * head chunks, B). A CTA takes up to 8 query heads of one key / value head and a range of the visible
+// keys; its 4 warps walk 16-key blocks independently, each through a cp.async ring of its own, with online softmax state in
+// registers. Products on mma.sync with register operands: the row tile of 16 is [map 1: 8 heads | map 2: 8 heads]; scores are
+// Q1 K1^T with map 2's rows zero plus Q2 K2^T with map 1's rows zero, so one accumulator holds both maps, and its layout is
+// the operand layout of the second product P V, which both maps share. P enters that product as a sum of two bf16 numbers
+// (value and rounding error), so the weights keep more than 16 bits. Slices are merged by the CTA that arrives last.
+constexpr int DD_WARPS = 4;
+constexpr int DD_KEYS = 16;       // keys per block
+constexpr int DD_HEADS = 8;       // query heads per CTA
+constexpr int DD_RING_LIMIT = 96 * 1024;
+
+struct DecodeParams {
+  const __nv_bfloat16* qkv;
+  long long ld;
+  const float *cos_t, *sin_t;
+  __nv_bfloat16 *kc, *vc, *out;
+  long long ldo;
+  const int *pos, *count;
+  const float* lam;
+  int H, G, dim, vdim, R, Smax, chunk;
+  float scale, eps, out_scale;
+  float* part;             // [B * G * head chunks][splits][16][vdim + 2]
+  unsigned int* counters;  // [B * G * head chunks], zero between launches
+  int stages;
+};
+
+__device__ __forceinline__ void dd_cp16(void* dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+}
+__device__ __forceinline__ void dd_mma(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+               : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ uint32_t dd_pack(float lo, float hi) {
+  uint32_t r;
+  asm("cvt.rn.bf16x2.f32 %0, %1, %2;" : "=r"(r) : "f"(hi), "f"(lo));
+  return r;
+}
+__device__ __forceinline__ float dd_lo(uint32_t v) { return __uint_as_float(v << 16); }
+__device__ __forceinline__ float dd_hi(uint32_t v) { return __uint_as_float(v & 0xffff0000u); }
+
+// bytes of one ring stage of one warp: 16 keys x 2 maps x KD pieces of 64 B, then 16 value rows of vdim + 8 elements
+__host__ __device__ constexpr int dd_stage_bytes(int kd, int vdim) { return DD_KEYS * 2 * kd * 64 + DD_KEYS * (vdim + 8) * 2; }
+
+// KD: 32-feature steps of a query / key row (dim <= 32 KD); VT: 8-feature tiles of a value row (vdim <= 8 VT)
+template <int KD, int VT>
+__global__ void __launch_bounds__(DD_WARPS * 32) diff_attn_decode_kernel(const DecodeParams p) {
+  extern __shared__ __align__(16) uint8_t smem[];
+  __shared__ __align__(16) __nv_bfloat16 sq[2][DD_HEADS][KD * 32];
+  __shared__ float sm[DD_WARPS][16], sl[DD_WARPS][16];
+  __shared__ unsigned int is_last;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, quad = lane >> 2, j = lane & 3;
+  const int per_g = p.H / p.G, hchunks = (per_g + DD_HEADS - 1) / DD_HEADS;
+  const int split = blockIdx.x, splits = gridDim.x, g = blockIdx.y / hchunks, b = blockIdx.z;
+  const int h0 = g * per_g + (blockIdx.y % hchunks) * DD_HEADS;  // first query head of this CTA
+  const int nh = min(DD_HEADS, (g + 1) * per_g - h0);
+  const int pos = p.pos[b];
+  if (p.count[b] <= 0 || pos < 0 || pos >= p.Smax) return;
+  const int first = p.chunk > 0 ? (pos / p.chunk) * p.chunk : 0;
+  const int len = pos + 1 - first;
+  const int blocks = (len + DD_KEYS - 1) / DD_KEYS;
+  const int blk0 = (int)((long long)split * blocks / splits), blk1 = (int)((long long)(split + 1) * blocks / splits);
+  const __nv_bfloat16* row = p.qkv + (long long)b * p.ld;
+  const __nv_bfloat16* kb = p.kc + ((long long)b * p.G + g) * 2 * p.Smax * p.dim;
+  const __nv_bfloat16* vb = p.vc + ((long long)b * p.G + g) * p.Smax * p.vdim;
+
+  // ---- rotated queries to shared memory; the CTAs with the last keys append the new key and value (the same data each) ----
+  const int half = p.dim / 2;  // dim is even
+  auto rotated = [&](const __nv_bfloat16* s, int e, float& y0, float& y1) {
+    const float x0 = __bfloat162float(s[0]), x1 = __bfloat162float(s[1]);
+    if (e < p.R) {
+      const float c = p.cos_t[(long long)pos * (p.R / 2) + e / 2], sn = p.sin_t[(long long)pos * (p.R / 2) + e / 2];
+      y0 = x0 * c - x1 * sn;
+      y1 = x1 * c + x0 * sn;
+    } else {
+      y0 = x0;
+      y1 = x1;
+    }
+  };
+  for (int i = threadIdx.x; i < 2 * DD_HEADS * KD * 16; i += blockDim.x) {
+    const int e = (i % (KD * 16)) * 2, hm = i / (KD * 16), m = hm / DD_HEADS, r = hm % DD_HEADS;
+    float y0 = 0.f, y1 = 0.f;
+    if (r < nh && e < p.dim) rotated(row + ((long long)(h0 + r) * 2 + m) * p.dim + e, e, y0, y1);
+    *reinterpret_cast<uint32_t*>(&sq[m][r][e]) = dd_pack(y0, y1);
+  }
+  if (split == splits - 1) {
+    for (int i = threadIdx.x; i < 2 * half; i += blockDim.x) {
+      const int m = i / half, e = (i % half) * 2;
+      float y0, y1;
+      rotated(row + ((long long)(p.H + g) * 2 + m) * p.dim + e, e, y0, y1);
+      *reinterpret_cast<uint32_t*>(p.kc + ((((long long)b * p.G + g) * 2 + m) * p.Smax + pos) * p.dim + e) = dd_pack(y0, y1);
+    }
+    const __nv_bfloat16* vsrc = row + (long long)(p.H + p.G) * 2 * p.dim + (long long)g * p.vdim;
+    __nv_bfloat16* vdst = p.vc + (((long long)b * p.G + g) * p.Smax + pos) * p.vdim;
+    for (int i = threadIdx.x; i < p.vdim; i += blockDim.x) vdst[i] = vsrc[i];
+    __threadfence();
+  }
+  __syncthreads();
+  uint4 q1[KD], q2[KD];
+#pragma unroll
+  for (int i = 0; i < KD; ++i) {
+    q1[i] = *reinterpret_cast<const uint4*>(&sq[0][quad][i * 32 + j * 8]);
+    q2[i] = *reinterpret_cast<const uint4*>(&sq[1][quad][i * 32 + j * 8]);
+  }
+  // ---- key blocks ---------------------------------------------------------------------------------------------------------
+  const int stage_bytes = dd_stage_bytes(KD, p.vdim), vld = p.vdim + 8;
+  uint8_t* ring = smem + (long long)warp * p.stages * stage_bytes;
+  const int mine = (blk1 - blk0 - warp + DD_WARPS - 1) / DD_WARPS;  // this warp's blocks: blk0 + warp, + DD_WARPS, ...
+  auto prefetch = [&](int n) {
+    if (n < mine) {
+      uint8_t* st = ring + (n % p.stages) * stage_bytes;
+      const int key0 = first + (blk0 + warp + n * DD_WARPS) * DD_KEYS;
+#pragma unroll
+      for (int m = 0; m < 2; ++m)
+#pragma unroll
+        for (int t = 0; t < 2; ++t) {
+          const int key = min(key0 + t * 8 + quad, pos);  // rows past the end repeat the last one and are masked
+          const __nv_bfloat16* src = kb + ((long long)m * p.Smax + key) * p.dim;
+#pragma unroll
+          for (int i = 0; i < KD; ++i) {
+            uint8_t* dst = st + (((m * 2 + t) * KD + i) * 32 + lane) * 16;
+            if (i * 32 + j * 8 < p.dim) dd_cp16(dst, src + i * 32 + j * 8);
+            else *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
+          }
+        }
+      uint8_t* sv = st + DD_KEYS * 2 * KD * 64;
+      const int pieces = p.vdim / 8;
+      for (int i = lane; i < DD_KEYS * pieces; i += 32) {
+        const int k = i / pieces, c = i % pieces;
+        dd_cp16(sv + (k * vld + c * 8) * 2, vb + (long long)min(key0 + k, pos) * p.vdim + c * 8);
+      }
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");  // possibly empty: keeps the group count per block fixed
+  };
+  float o[VT][4];
+#pragma unroll
+  for (int t = 0; t < VT; ++t)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) o[t][e] = 0.f;
+  float mx[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};  // rows quad (map 1) and quad + 8 (map 2)
+  const float sc = p.scale * 1.4426950408889634f;
+  for (int n = 0; n < p.stages - 1; ++n) prefetch(n);
+  for (int n = 0; n < mine; ++n) {
+    prefetch(n + p.stages - 1);
+    if (p.stages == 2) asm volatile("cp.async.wait_group 1;" ::: "memory");
+    else asm volatile("cp.async.wait_group 2;" ::: "memory");
+    __syncwarp();
+    const uint8_t* st = ring + (n % p.stages) * stage_bytes;
+    const int key0 = first + (blk0 + warp + n * DD_WARPS) * DD_KEYS;
+    float s[2][4];
+#pragma unroll
+    for (int t = 0; t < 2; ++t) {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) s[t][e] = 0.f;
+#pragma unroll
+      for (int i = 0; i < KD; ++i) {
+        const uint4 k1 = *reinterpret_cast<const uint4*>(st + ((t * KD + i) * 32 + lane) * 16);
+        const uint4 k2 = *reinterpret_cast<const uint4*>(st + (((2 + t) * KD + i) * 32 + lane) * 16);
+        dd_mma(s[t], q1[i].x, 0u, q1[i].y, 0u, k1.x, k1.y);
+        dd_mma(s[t], 0u, q2[i].x, 0u, q2[i].y, k2.x, k2.y);
+        dd_mma(s[t], q1[i].z, 0u, q1[i].w, 0u, k1.z, k1.w);
+        dd_mma(s[t], 0u, q2[i].z, 0u, q2[i].w, k2.z, k2.w);
+      }
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        s[t][e] = key0 + t * 8 + 2 * j + (e & 1) <= pos ? s[t][e] * sc : -INFINITY;
+    }
+    float alpha[2];
+#pragma unroll
+    for (int m = 0; m < 2; ++m) {
+      float v = fmaxf(fmaxf(s[0][2 * m], s[0][2 * m + 1]), fmaxf(s[1][2 * m], s[1][2 * m + 1]));
+      v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, 1));
+      v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, 2));
+      const float m_new = fmaxf(mx[m], v);  // finite: the first key of a block is always visible
+      alpha[m] = exp2f(mx[m] - m_new);
+      mx[m] = m_new;
+      float sum = 0.f;
+#pragma unroll
+      for (int t = 0; t < 2; ++t)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          s[t][2 * m + e] = exp2f(s[t][2 * m + e] - m_new);
+          sum += s[t][2 * m + e];
+        }
+      l[m] = l[m] * alpha[m] + sum;  // this lane's share of the row sum
+    }
+    uint32_t ph[4], pl[4];
+#pragma unroll
+    for (int t = 0; t < 2; ++t)
+#pragma unroll
+      for (int m = 0; m < 2; ++m) {
+        const float x = s[t][2 * m], y = s[t][2 * m + 1];
+        const uint32_t hi = dd_pack(x, y);
+        ph[2 * t + m] = hi;
+        pl[2 * t + m] = dd_pack(x - dd_lo(hi), y - dd_hi(hi));
+      }
+    const uint32_t sv = (uint32_t)__cvta_generic_to_shared(st + DD_KEYS * 2 * KD * 64);
+    const uint32_t vaddr = sv + (((lane & 7) + ((lane >> 3) & 1) * 8) * vld + (lane >> 4) * 8) * 2;
+#pragma unroll
+    for (int t = 0; t < VT; t += 2) {
+      if (t * 8 < p.vdim) {
+        uint32_t v0, v1, v2, v3;  // key pairs of value tiles t (v0, v1) and t + 1 (v2, v3)
+        asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
+                     : "=r"(v0), "=r"(v1), "=r"(v2), "=r"(v3)
+                     : "r"(vaddr + t * 16));
+#pragma unroll
+        for (int u = 0; u < 2; ++u) {
+          o[t + u][0] *= alpha[0];
+          o[t + u][1] *= alpha[0];
+          o[t + u][2] *= alpha[1];
+          o[t + u][3] *= alpha[1];
+        }
+        dd_mma(o[t], ph[0], ph[1], ph[2], ph[3], v0, v1);
+        dd_mma(o[t + 1], ph[0], ph[1], ph[2], ph[3], v2, v3);
+        dd_mma(o[t], pl[0], pl[1], pl[2], pl[3], v0, v1);
+        dd_mma(o[t + 1], pl[0], pl[1], pl[2], pl[3], v2, v3);
+      }
+    }
+    __syncwarp();  // every lane has read the stage before it is refilled
+  }
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
+#pragma unroll
+  for (int m = 0; m < 2; ++m) {
+    l[m] += __shfl_xor_sync(0xffffffffu, l[m], 1);
+    l[m] += __shfl_xor_sync(0xffffffffu, l[m], 2);
+    if (j == 0) {
+      sm[warp][quad + 8 * m] = mx[m];
+      sl[warp][quad + 8 * m] = l[m];
+    }
+  }
+  __syncthreads();  // all rings are idle: their memory holds the warps' outputs from here on
+  float* so = reinterpret_cast<float*>(smem);  // [DD_WARPS][16][vdim]
+#pragma unroll
+  for (int t = 0; t < VT; ++t) {
+    if (t * 8 < p.vdim) {
+      float* d = so + ((long long)warp * 16 + quad) * p.vdim + t * 8 + 2 * j;
+      d[0] = o[t][0];
+      d[1] = o[t][1];
+      d += 8 * p.vdim;
+      d[0] = o[t][2];
+      d[1] = o[t][3];
+    }
+  }
+  __syncthreads();
+  // ---- merge of the warps; the slice's result goes to `part`, or stays here when there is one slice ------------------------
+  __shared__ float fm[16], fl[16];
+  const long long unit = (long long)b * gridDim.y + blockIdx.y;
+  const int pw = p.vdim + 2;
+  float* mypart = p.part + (unit * splits + split) * 16 * pw;
+  if (threadIdx.x < 16) {
+    const int r = threadIdx.x;
+    float m = -INFINITY, ll = 0.f;
+    for (int w = 0; w < DD_WARPS; ++w) m = fmaxf(m, sm[w][r]);
+    for (int w = 0; w < DD_WARPS; ++w) ll += sm[w][r] == -INFINITY ? 0.f : sl[w][r] * exp2f(sm[w][r] - m);
+    fm[r] = m;
+    fl[r] = ll;
+    if (splits > 1) {
+      __stcg(mypart + r * pw, m);
+      __stcg(mypart + r * pw + 1, ll);
+    }
+  }
+  __syncthreads();
+  for (int i = threadIdx.x; i < 16 * p.vdim; i += blockDim.x) {
+    const int r = i / p.vdim, c = i % p.vdim;
+    if ((r & 7) >= nh) continue;
+    float acc = 0.f;
+#pragma unroll
+    for (int w = 0; w < DD_WARPS; ++w)
+      acc += sm[w][r] == -INFINITY ? 0.f : so[((long long)w * 16 + r) * p.vdim + c] * exp2f(sm[w][r] - fm[r]);
+    if (splits > 1) __stcg(mypart + r * pw + 2 + c, acc);
+    else so[(long long)r * p.vdim + c] = acc;  // warp 0's copy: read and written by this thread only
+  }
+  if (splits > 1) {
+    __threadfence();
+    __syncthreads();
+    if (threadIdx.x == 0) is_last = atomicAdd(p.counters + unit, 1u) == (unsigned int)splits - 1;
+    __syncthreads();
+    if (!is_last) return;
+    __threadfence();
+    const float* parts = p.part + unit * splits * 16 * pw;
+    if (threadIdx.x < 16) {
+      const int r = threadIdx.x;
+      float m = -INFINITY, ll = 0.f;
+      for (int k = 0; k < splits; ++k) m = fmaxf(m, __ldcg(parts + ((long long)k * 16 + r) * pw));
+      for (int k = 0; k < splits; ++k) {
+        const float mk = __ldcg(parts + ((long long)k * 16 + r) * pw);
+        ll += mk == -INFINITY ? 0.f : __ldcg(parts + ((long long)k * 16 + r) * pw + 1) * exp2f(mk - m);
+      }
+      fm[r] = m;
+      fl[r] = ll;
+    }
+    __syncthreads();
+    for (int i = threadIdx.x; i < 16 * p.vdim; i += blockDim.x) {
+      const int r = i / p.vdim, c = i % p.vdim;
+      if ((r & 7) >= nh) continue;
+      float acc = 0.f;
+      for (int k = 0; k < splits; ++k) {
+        const float* src = parts + ((long long)k * 16 + r) * pw;
+        const float mk = __ldcg(src);
+        if (mk != -INFINITY) acc += __ldcg(src + 2 + c) * exp2f(mk - fm[r]);
+      }
+      so[(long long)r * p.vdim + c] = acc;
+    }
+    if (threadIdx.x == 0) p.counters[unit] = 0;
+  }
+  __syncthreads();
+  // ---- a_1 - lambda a_2, divided by its root mean square: one warp per head -------------------------------------------------
+  const float lambda = *p.lam;
+  for (int r = warp; r < nh; r += DD_WARPS) {
+    const float i1 = 1.f / fl[r], i2 = lambda / fl[r + 8];
+    float ss = 0.f;
+    for (int c = lane; c < p.vdim; c += 32) {
+      const float v = so[(long long)r * p.vdim + c] * i1 - so[(long long)(r + 8) * p.vdim + c] * i2;
+      so[(long long)r * p.vdim + c] = v;
+      ss += v * v;
+    }
+    ss = xl_warp_sum(ss);
+    const float f = p.out_scale / sqrtf(ss / p.vdim + p.eps);
+    for (int c = lane; c < p.vdim; c += 32)
+      p.out[(long long)b * p.ldo + (long long)(h0 + r) * p.vdim + c] = __float2bfloat16_rn(so[(long long)r * p.vdim + c] * f);
+  }
+}
+
+template <int KD, int VT> int dd_launch(DecodeParams p, int B, int splits, cudaStream_t s) {
+  const int stage = dd_stage_bytes(KD, p.vdim) * DD_WARPS;
+  p.stages = 3 * stage <= DD_RING_LIMIT ? 3 : 2;
+  int bytes = p.stages * stage;
+  const int merge = DD_WARPS * 16 * p.vdim * 4;
+  if (bytes < merge) bytes = merge;
+  static int configured = 0;
+  if (configured < bytes) {
+    const cudaError_t e = cudaFuncSetAttribute(diff_attn_decode_kernel<KD, VT>, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
+    if (e != cudaSuccess) return (int)e;
+    configured = bytes;
+  }
+  const int hchunks = (p.H / p.G + DD_HEADS - 1) / DD_HEADS;
+  diff_attn_decode_kernel<KD, VT><<<dim3(splits, p.G * hchunks, B), DD_WARPS * 32, bytes, s>>>(p);
+  return (int)cudaGetLastError();
+}
+
 }  // namespace
 
 // qkv: (B*T_len, ld) as described above, q rotated in place. cos / sin tables (Smax, R/2) fp32 (null when R == 0).
@@ -181,4 +524,31 @@ XL_API int xl_diff_attn_general(const void* q, long long ldq, const void* kc, co
                                                               out_scale);
   });
   return (int)cudaGetLastError();
+}
+
+// One token per sequence (rows of qkv = sequences), bf16. dim, vdim multiples of 8, dim <= 128, vdim <= 256, ld a multiple of
+// 8. The new key and value are rotated / appended by the kernel; q is not modified. part: B * G * ceil(H/G/8) * splits * 16 *
+// (vdim + 2) floats; counters: B * G * ceil(H/G/8) zero-initialised words (left zeroed). Sequences with count 0 are skipped.
+XL_API int xl_diff_attn_decode(const void* qkv, long long ld, const float* cos_t, const float* sin_t, void* kc, void* vc,
+                               void* out, long long ldo, const int* pos, const int* count, const float* lam, int B, int H, int G,
+                               int dim, int vdim, int R, int Smax, int chunk, float scale, float eps, float out_scale,
+                               int splits, float* part, unsigned int* counters, cudaStream_t s) {
+  if (B < 1 || B > 65535 || G < 1 || H % G || H > 4096 || dim < 8 || dim > 128 || dim % 8 || vdim < 8 || vdim > 256 || vdim % 8 ||
+      R < 0 || R > dim || (R & 1) || Smax < 1 || chunk < 0 || splits < 1 || splits > 1024 || (ld % 8))
+    return -1;
+  if (((uintptr_t)qkv & 15) || ((uintptr_t)kc & 15) || ((uintptr_t)vc & 15) || (R > 0 && (!cos_t || !sin_t))) return -1;
+  if (splits > 1 && (!part || !counters)) return -1;
+  DecodeParams p = {};
+  p.qkv = (const __nv_bfloat16*)qkv; p.ld = ld; p.cos_t = cos_t; p.sin_t = sin_t;
+  p.kc = (__nv_bfloat16*)kc; p.vc = (__nv_bfloat16*)vc; p.out = (__nv_bfloat16*)out; p.ldo = ldo;
+  p.pos = pos; p.count = count; p.lam = lam; p.H = H; p.G = G; p.dim = dim; p.vdim = vdim; p.R = R; p.Smax = Smax;
+  p.chunk = chunk; p.scale = scale; p.eps = eps; p.out_scale = out_scale; p.part = part; p.counters = counters;
+#define XL_DD(KD)                                       \
+  if (vdim <= 64) return dd_launch<KD, 8>(p, B, splits, s);   \
+  if (vdim <= 128) return dd_launch<KD, 16>(p, B, splits, s); \
+  return dd_launch<KD, 32>(p, B, splits, s);
+  if (dim <= 32) { XL_DD(1) }
+  if (dim <= 64) { XL_DD(2) }
+  XL_DD(4)
+#undef XL_DD
 }

@@ -1,0 +1,352 @@
+// Linear layers of the decoding path, bf16 weights, M <= 16 rows: C[M, N] = a[M, K] * w[N, K]^T, the weights streamed once.
+// What follows the product in a layer happens in the epilogue, on the fp32 sums:
+//   store      C as bf16 or fp32
+//   residual   x += mult * C (+ table[token]) on the fp32 residual stream, h = DyT(x) for the next layer
+//   swiglu     weight rows [gate | up]: y = silu(gate) * up
+//   min_gru    weight rows [z | u | g], one row per sequence: one step of the recurrence on the fp32 state
+//
+// The product is bandwidth-bound (at most 16 multiply-adds per weight), so it uses `mma.sync.m16n8k16` with operands from
+// registers: each lane copies 32 contiguous bytes of a weight row through a per-warp cp.async ring and feeds them to four
+// MMAs. (Any assignment of k indices to the k slots of an MMA is valid as long as both operands agree.)
+//
+// Work = (column tiles) x (K chunks of 64), tile-major, cut into equal contiguous ranges, one per CTA, so the grid fits the
+// machine and not the problem. A tile shared by several CTAs is finished by the one that arrives last: every CTA leaves its
+// partial sums in a slot of its own and the finisher adds the slots in CTA order, so results do not depend on timing.
+// Nobody waits for anybody. An epilogue that combines several weight rows per output channel (swiglu, min_gru) takes them
+// into one tile: a tile is PARTS groups of CH channels, group p starting at weight row p * N / PARTS.
+#include "common.cuh"
+
+#include <math.h>
+
+namespace {
+
+constexpr int SM_WARPS = 4;
+constexpr int SM_KC = 64;       // k values per chunk (16 per lane)
+constexpr int SM_STAGES = 2;
+constexpr int SM_CTAS_PER_SM = 2;
+
+enum SmMode : int { SM_STORE = 0, SM_RESIDUAL = 1, SM_SWIGLU = 2, SM_MINGRU = 3 };
+
+template <int MODE> struct SmTile {
+  static constexpr int PARTS = MODE == SM_SWIGLU ? 2 : (MODE == SM_MINGRU ? 3 : 1);
+  static constexpr int CH = MODE == SM_SWIGLU ? 32 : (MODE == SM_MINGRU ? 16 : 64);  // channels per tile
+  static constexpr int COLS = PARTS * CH;
+  static constexpr int NT = COLS / 8;
+  static constexpr int STAGE = (NT + 2) * 2 * 32;  // uint4: NT weight pieces and two activation rows, 2 x 16 bytes a lane
+  static constexpr int RING_BYTES = SM_WARPS * SM_STAGES * STAGE * 16;
+};
+
+struct SmParams {
+  const __nv_bfloat16* a;
+  long long lda;
+  const __nv_bfloat16* w;  // (N, K), contiguous
+  int M, N, K;
+  // store / swiglu / min_gru
+  void* y;
+  long long ldy;
+  int y_f32;
+  // residual
+  float* x;
+  float mult;
+  const int* tokens;
+  const __nv_bfloat16* table;
+  int vocab;
+  const float *alpha, *nw, *nb;
+  __nv_bfloat16* h;
+  // min_gru
+  const float *bz, *bu;
+  float* state;
+  const int *pos, *count;
+  // split-K scratch
+  float* slots;            // [grid][2][16 * COLS]
+  unsigned int* counters;  // one per tile, zero between launches
+};
+
+__device__ __forceinline__ void cp_async16(uint4* dst, const void* src, bool on) {
+  const int bytes = on ? 16 : 0;  // 0: the destination is zero-filled
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src),
+               "r"(bytes)
+               : "memory");
+}
+__device__ __forceinline__ void mma_bf16(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0,
+                                         uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+               : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ float sigmoid_f(float v) { return 1.f / (1.f + expf(-v)); }
+__device__ __forceinline__ float silu_f(float v) { return v / (1.f + expf(-v)); }
+
+template <int MODE>
+__device__ __forceinline__ void sm_epilogue(const SmParams& p, int r, int c, const float (&v)[SmTile<MODE>::PARTS], int channels) {
+  if (MODE == SM_STORE) {
+    if (p.y_f32) ((float*)p.y)[(long long)r * p.ldy + c] = v[0];
+    else ((__nv_bfloat16*)p.y)[(long long)r * p.ldy + c] = __float2bfloat16_rn(v[0]);
+  } else if (MODE == SM_RESIDUAL) {
+    float* xp = p.x + (long long)r * channels + c;
+    float s = *xp + p.mult * v[0];
+    if (p.table) {
+      const int t = min(max(p.tokens[r], 0), p.vocab - 1);
+      s += __bfloat162float(p.table[(long long)t * channels + c]);
+    }
+    *xp = s;
+    if (p.alpha) p.h[(long long)r * channels + c] = __float2bfloat16_rn(tanhf(*p.alpha * s) * p.nw[c] + p.nb[c]);
+  } else if (MODE == SM_SWIGLU) {
+    ((__nv_bfloat16*)p.y)[(long long)r * p.ldy + c] = __float2bfloat16_rn(silu_f(v[0]) * v[SmTile<MODE>::PARTS - 1]);
+  } else {
+    const float z = sigmoid_f(v[0] + p.bz[c]);
+    const float u = v[1 % SmTile<MODE>::PARTS] + p.bu[c];
+    const float cand = u >= 0.f ? u + 0.5f : sigmoid_f(u);
+    float* sp = p.state + (long long)r * channels + c;
+    float s = p.pos[r] > 0 ? *sp : 0.f;
+    if (p.count[r] > 0) {
+      s = (1.f - z) * s + z * cand;
+      *sp = s;
+    }
+    ((__nv_bfloat16*)p.y)[(long long)r * p.ldy + c] = __float2bfloat16_rn(s * silu_f(v[SmTile<MODE>::PARTS - 1]));
+  }
+}
+
+__device__ __forceinline__ long long sm_begin(long long total, int cta, int grid) { return total * cta / grid; }
+
+template <int MODE>
+__global__ void __launch_bounds__(SM_WARPS * 32, SM_CTAS_PER_SM) linear_small_m_kernel(const SmParams p) {
+  using L = SmTile<MODE>;
+  constexpr int NT = L::NT, COLS = L::COLS, CH = L::CH, PARTS = L::PARTS;
+  extern __shared__ uint4 ring_all[];
+  __shared__ float red[SM_WARPS][16][COLS + 1];
+  __shared__ unsigned int finish;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int quad = lane >> 2, j = lane & 3;
+  const int channels = p.N / PARTS;
+  const int chunks = (p.K + SM_KC - 1) / SM_KC;
+  const int n_tiles = (channels + CH - 1) / CH;
+  const long long total = (long long)n_tiles * chunks;
+  const int grid = (int)gridDim.x;
+  long long item = sm_begin(total, blockIdx.x, grid);
+  const long long item_end = sm_begin(total, blockIdx.x + 1, grid);
+  const int first_tile = (int)(item / chunks);
+  uint4* ring = ring_all + warp * (SM_STAGES * L::STAGE);
+
+  auto prefetch = [&](int tile, int ch, int buf) {
+    const int k0 = ch * SM_KC + j * 16;
+    uint4* dst = ring + buf * L::STAGE + lane;
+#pragma unroll
+    for (int t = 0; t < NT; ++t) {
+      const int col = t * 8 + quad, part = col / CH, c = tile * CH + col % CH;
+      const bool row_on = c < channels;
+      const __nv_bfloat16* src = p.w + ((long long)part * channels + (row_on ? c : 0)) * p.K;
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const bool on = row_on && k0 + e * 8 < p.K;
+        cp_async16(dst + (t * 2 + e) * 32, src + (on ? k0 + e * 8 : 0), on);
+      }
+    }
+#pragma unroll
+    for (int hi = 0; hi < 2; ++hi) {
+      const int r = quad + hi * 8;
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const bool on = r < p.M && k0 + e * 8 < p.K;
+        cp_async16(dst + ((NT + hi) * 2 + e) * 32, p.a + (on ? (long long)r * p.lda + k0 + e * 8 : 0), on);
+      }
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+
+  int buf = 0;
+  bool have = false;  // ring[buf] holds (or is receiving) this warp's first chunk of the current tile
+  while (item < item_end) {
+    const int tile = (int)(item / chunks);
+    const int c0 = (int)(item - (long long)tile * chunks);
+    const int c1 = (int)min((long long)chunks, c0 + (item_end - item));
+    float acc[NT][4];
+#pragma unroll
+    for (int t = 0; t < NT; ++t)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc[t][e] = 0.f;
+    if (!have && c0 + warp < c1) prefetch(tile, c0 + warp, buf);
+    have = false;
+    for (int ch = c0 + warp; ch < c1; ch += SM_WARPS) {
+      // request the chunk after this one: the next of this tile, or this warp's first of the next tile
+      bool next = false;
+      if (ch + SM_WARPS < c1) {
+        prefetch(tile, ch + SM_WARPS, buf ^ 1);
+        next = true;
+      } else {
+        const long long nit = item + (c1 - c0);
+        if (nit < item_end) {
+          const int nc1 = (int)min((long long)chunks, item_end - nit);  // the next tile starts at its first chunk
+          if (warp < nc1) {
+            prefetch(tile + 1, warp, buf ^ 1);
+            next = have = true;
+          }
+        }
+      }
+      if (next) asm volatile("cp.async.wait_group 1;" ::: "memory");
+      else asm volatile("cp.async.wait_group 0;" ::: "memory");
+      const uint4* src = ring + buf * L::STAGE + lane;  // every lane reads back the pieces it copied itself
+      buf ^= 1;
+      uint32_t lo[8], hi[8];
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        *reinterpret_cast<uint4*>(lo + 4 * e) = src[(NT * 2 + e) * 32];
+        *reinterpret_cast<uint4*>(hi + 4 * e) = src[((NT + 1) * 2 + e) * 32];
+      }
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        uint4 w[NT];
+#pragma unroll
+        for (int t = 0; t < NT; ++t) w[t] = src[(t * 2 + e) * 32];
+#pragma unroll
+        for (int s = 0; s < 2; ++s)
+#pragma unroll
+          for (int t = 0; t < NT; ++t) {
+            const uint32_t* ww = reinterpret_cast<const uint32_t*>(&w[t]);
+            mma_bf16(acc[t], lo[4 * e + 2 * s], hi[4 * e + 2 * s], lo[4 * e + 2 * s + 1], hi[4 * e + 2 * s + 1], ww[2 * s],
+                     ww[2 * s + 1]);
+          }
+      }
+    }
+    __syncthreads();  // readers of the previous tile are done with `red`
+#pragma unroll
+    for (int t = 0; t < NT; ++t) {
+      red[warp][quad][t * 8 + 2 * j] = acc[t][0];
+      red[warp][quad][t * 8 + 2 * j + 1] = acc[t][1];
+      red[warp][quad + 8][t * 8 + 2 * j] = acc[t][2];
+      red[warp][quad + 8][t * 8 + 2 * j + 1] = acc[t][3];
+    }
+    __syncthreads();
+    const bool whole = c1 - c0 == chunks;
+    bool finishing = whole;
+    if (!whole) {
+      float* slot = p.slots + ((long long)blockIdx.x * 2 + (tile == first_tile ? 0 : 1)) * (16 * COLS);
+      for (int i = threadIdx.x; i < p.M * COLS; i += blockDim.x) {
+        const int r = i / COLS, col = i % COLS;
+        float s = 0.f;
+#pragma unroll
+        for (int w = 0; w < SM_WARPS; ++w) s += red[w][r][col];
+        __stcg(slot + i, s);
+      }
+      __threadfence();
+      __syncthreads();
+      if (threadIdx.x == 0)
+        finish = atomicAdd(p.counters + tile, (unsigned int)(c1 - c0)) + (unsigned int)(c1 - c0) == (unsigned int)chunks;
+      __syncthreads();
+      finishing = finish != 0;
+      if (finishing) __threadfence();
+    }
+    if (finishing) {
+      // CTAs that share the tile, in order
+      int cta0 = blockIdx.x, cta1 = blockIdx.x;
+      if (!whole) {
+        const long long lo_item = (long long)tile * chunks, hi_item = lo_item + chunks - 1;
+        cta0 = (int)(lo_item * grid / total);
+        while (cta0 > 0 && sm_begin(total, cta0, grid) > lo_item) --cta0;
+        while (sm_begin(total, cta0 + 1, grid) <= lo_item) ++cta0;
+        cta1 = cta0;
+        while (sm_begin(total, cta1 + 1, grid) <= hi_item) ++cta1;
+      }
+      for (int i = threadIdx.x; i < p.M * CH; i += blockDim.x) {
+        const int r = i / CH, cc = i % CH, c = tile * CH + cc;
+        if (c >= channels) continue;
+        float v[PARTS];
+#pragma unroll
+        for (int q = 0; q < PARTS; ++q) {
+          const int col = q * CH + cc;
+          float s = 0.f;
+          if (whole) {
+#pragma unroll
+            for (int w = 0; w < SM_WARPS; ++w) s += red[w][r][col];
+          } else {
+            for (int k = cta0; k <= cta1; ++k) {
+              const int which = (int)(sm_begin(total, k, grid) / chunks) == tile ? 0 : 1;
+              s += __ldcg(p.slots + ((long long)k * 2 + which) * (16 * COLS) + r * COLS + col);
+            }
+          }
+          v[q] = s;
+        }
+        sm_epilogue<MODE>(p, r, c, v, channels);
+      }
+      if (!whole && threadIdx.x == 0) p.counters[tile] = 0;
+    }
+    item += c1 - c0;
+  }
+}
+
+template <int MODE> int sm_launch(const SmParams& p, int sms, int max_tiles, cudaStream_t s) {
+  using L = SmTile<MODE>;
+  if (p.N % L::PARTS) return -1;
+  const int channels = p.N / L::PARTS, chunks = (p.K + SM_KC - 1) / SM_KC, n_tiles = (channels + L::CH - 1) / L::CH;
+  if (n_tiles > max_tiles) return -1;
+  static bool configured = false;
+  if (!configured) {
+    const cudaError_t e =
+        cudaFuncSetAttribute(linear_small_m_kernel<MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, L::RING_BYTES);
+    if (e != cudaSuccess) return (int)e;
+    configured = true;
+  }
+  long long grid = (long long)SM_CTAS_PER_SM * sms;
+  const long long total = (long long)n_tiles * chunks;
+  if (grid > total) grid = total;
+  linear_small_m_kernel<MODE><<<(int)grid, SM_WARPS * 32, L::RING_BYTES, s>>>(p);
+  return (int)cudaGetLastError();
+}
+
+int sm_check(const void* a, long long lda, const void* w, int M, int N, int K, const float* slots, const unsigned int* counters) {
+  if (M < 1 || M > 16 || N < 1 || K < 8 || (K % 8) || (lda % 8) || lda < K) return -1;
+  if (((uintptr_t)a & 15) || ((uintptr_t)w & 15) || !slots || !counters) return -1;
+  return 0;
+}
+
+}  // namespace
+
+// Floats of `slots` for a device with `sms` SMs; `counters` needs `max_tiles` zero-initialised words (left zeroed).
+XL_API int xl_linear_small_m_slots(int sms) { return SM_CTAS_PER_SM * sms * 2 * 16 * 64; }
+
+// All: a (M, K) bf16 with row stride lda (a multiple of 8), w (N, K) bf16 contiguous, M <= 16, K a multiple of 8; returns -1
+// for arguments the kernel does not take. y (M, N) with row stride ldy, bf16 or fp32.
+XL_API int xl_linear_small_m(const void* a, long long lda, const void* w, void* y, long long ldy, int y_f32, int M, int N, int K,
+                             float* slots, unsigned int* counters, int max_tiles, int sms, cudaStream_t s) {
+  if (sm_check(a, lda, w, M, N, K, slots, counters) || !y) return -1;
+  SmParams p = {};
+  p.a = (const __nv_bfloat16*)a; p.lda = lda; p.w = (const __nv_bfloat16*)w; p.M = M; p.N = N; p.K = K;
+  p.y = y; p.ldy = ldy; p.y_f32 = y_f32; p.slots = slots; p.counters = counters;
+  return sm_launch<SM_STORE>(p, sms, max_tiles, s);
+}
+
+// x (M, N) fp32 += mult * a w^T (+ table[tokens]); with alpha, h (M, N) bf16 = tanh(alpha x) nw + nb.
+XL_API int xl_linear_small_m_residual(const void* a, long long lda, const void* w, float* x, float mult, const int* tokens,
+                                      const void* table, int vocab, const float* alpha, const float* nw, const float* nb,
+                                      void* h, int M, int N, int K, float* slots, unsigned int* counters, int max_tiles, int sms,
+                                      cudaStream_t s) {
+  if (sm_check(a, lda, w, M, N, K, slots, counters) || !x || (table && (!tokens || vocab < 1)) || (alpha && (!nw || !nb || !h)))
+    return -1;
+  SmParams p = {};
+  p.a = (const __nv_bfloat16*)a; p.lda = lda; p.w = (const __nv_bfloat16*)w; p.M = M; p.N = N; p.K = K;
+  p.x = x; p.mult = mult; p.tokens = tokens; p.table = (const __nv_bfloat16*)table; p.vocab = vocab;
+  p.alpha = alpha; p.nw = nw; p.nb = nb; p.h = (__nv_bfloat16*)h; p.slots = slots; p.counters = counters;
+  return sm_launch<SM_RESIDUAL>(p, sms, max_tiles, s);
+}
+
+// w rows [gate | up] (2F, K); y (M, F) bf16 contiguous.
+XL_API int xl_linear_small_m_swiglu(const void* a, long long lda, const void* w, void* y, int M, int F, int K, float* slots,
+                                    unsigned int* counters, int max_tiles, int sms, cudaStream_t s) {
+  if (sm_check(a, lda, w, M, 2 * F, K, slots, counters) || !y) return -1;
+  SmParams p = {};
+  p.a = (const __nv_bfloat16*)a; p.lda = lda; p.w = (const __nv_bfloat16*)w; p.M = M; p.N = 2 * F; p.K = K;
+  p.y = y; p.ldy = F; p.slots = slots; p.counters = counters;
+  return sm_launch<SM_SWIGLU>(p, sms, max_tiles, s);
+}
+
+// w rows [z | u | g] (3W, K); row r is the next token of sequence r: state (M, W) fp32 advances where count[r] > 0 and starts
+// from zero at pos[r] == 0; y (M, W) bf16 contiguous.
+XL_API int xl_linear_small_m_min_gru(const void* a, long long lda, const void* w, const float* bz, const float* bu, float* state,
+                                     const int* pos, const int* count, void* y, int M, int W, int K, float* slots,
+                                     unsigned int* counters, int max_tiles, int sms, cudaStream_t s) {
+  if (sm_check(a, lda, w, M, 3 * W, K, slots, counters) || !y || !state || !bz || !bu || !pos || !count) return -1;
+  SmParams p = {};
+  p.a = (const __nv_bfloat16*)a; p.lda = lda; p.w = (const __nv_bfloat16*)w; p.M = M; p.N = 3 * W; p.K = K;
+  p.y = y; p.ldy = W; p.bz = bz; p.bu = bu; p.state = state; p.pos = pos; p.count = count; p.slots = slots; p.counters = counters;
+  return sm_launch<SM_MINGRU>(p, sms, max_tiles, s);
+}

@@ -2,8 +2,8 @@
 32-bit models use plain fp32 matrix products (never a reduced-precision matrix mode) and the same kernels for the rest."""
 import torch
 
-from ..xl.opdef import OPS, native
-from .native import (_CODE, _c_f, _c_int, _c_ll, _c_p, _check, _count, _ok, _sig, _stream, gemm)
+from ..xl.opdef import native
+from .native import (_CODE, _c_f, _c_int, _c_ll, _c_p, _check, _count, _ok, _sig, _sms, _stream, gemm)
 
 _stream_dyt = _sig("xl_stream_dyt", _c_p, _c_p, _c_f, _c_p, _c_p, _c_int, _c_p, _c_p, _c_p, _c_p, _c_ll, _c_int, _c_int, _c_p)
 _select_dyt = _sig("xl_select_dyt", _c_p, _c_p, _c_int, _c_int, _c_ll, _c_p, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int, _c_p)
@@ -14,6 +14,48 @@ _rope_append = _sig("xl_diff_rope_append", _c_p, _c_ll, _c_p, _c_p, _c_p, _c_p, 
                     _c_int, _c_int, _c_int, _c_int, _c_int, _c_p)
 _diff_general = _sig("xl_diff_attn_general", _c_p, _c_ll, _c_p, _c_p, _c_p, _c_ll, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int,
                      _c_int, _c_int, _c_int, _c_int, _c_int, _c_f, _c_f, _c_f, _c_int, _c_p)
+_diff_decode = _sig("xl_diff_attn_decode", _c_p, _c_ll, _c_p, _c_p, _c_p, _c_p, _c_p, _c_ll, _c_p, _c_p, _c_p, _c_int, _c_int,
+                    _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_f, _c_f, _c_f, _c_int, _c_p, _c_p, _c_p)
+_small_m_slots = _sig("xl_linear_small_m_slots", _c_int)
+_SMALL_TAIL = (_c_int, _c_int, _c_int, _c_p, _c_p, _c_int, _c_int, _c_p)
+_small_store = _sig("xl_linear_small_m", _c_p, _c_ll, _c_p, _c_p, _c_ll, _c_int, *_SMALL_TAIL)
+_small_residual = _sig("xl_linear_small_m_residual", _c_p, _c_ll, _c_p, _c_p, _c_f, _c_p, _c_p, _c_int, _c_p, _c_p, _c_p, _c_p,
+                       *_SMALL_TAIL)
+_small_swiglu = _sig("xl_linear_small_m_swiglu", _c_p, _c_ll, _c_p, _c_p, *_SMALL_TAIL)
+_small_min_gru = _sig("xl_linear_small_m_min_gru", _c_p, _c_ll, _c_p, _c_p, _c_p, _c_p, _c_p, _c_p, _c_p, *_SMALL_TAIL)
+
+_MAX_TILES = 1 << 14  # column tiles the split-K counters of the small-M kernel cover
+_SCRATCH = {}
+
+
+def _scratch(device):
+    """Per-device scratch of the decoding kernels: partial sums, and counters that every launch leaves at zero. Allocated
+    once at its final size, since captured graphs keep the addresses."""
+    idx = device.index or 0
+    if idx not in _SCRATCH:
+        _SCRATCH[idx] = (torch.empty(_small_m_slots(_sms(device)), dtype=torch.float32, device=device),
+                         torch.zeros(_MAX_TILES, dtype=torch.int32, device=device),
+                         torch.zeros(1 << 16, dtype=torch.int32, device=device))
+    return _SCRATCH[idx]
+
+
+def _small(a, weight) -> bool:
+    """Whether the small-M kernels take this product."""
+    return (a.dtype == torch.bfloat16 and weight.dtype == torch.bfloat16 and a.shape[0] <= 16 and a.is_cuda
+            and a.stride(1) == 1 and weight.is_contiguous() and a.shape[1] % 8 == 0)
+
+
+def _small_tail(a, rows, weight):
+    slots, counters, _ = _scratch(a.device)
+    return (a.shape[0], rows, weight.shape[1], slots.data_ptr(), counters.data_ptr(), _MAX_TILES, _sms(a.device), _stream())
+
+
+def _small_ok(rc, name) -> bool:
+    if rc == -1:
+        return False
+    _check(rc, name)
+    _count(name)
+    return True
 
 
 def _ptr(t):
@@ -33,6 +75,12 @@ def product(a, weight, out_dtype=None):
     sizes it does not take and for 32-bit models."""
     out_dtype = out_dtype or a.dtype
     if a.dtype != torch.float32:
+        if _small(a, weight) and out_dtype in (torch.bfloat16, torch.float32):
+            y = torch.empty((a.shape[0], weight.shape[0]), dtype=out_dtype, device=a.device)
+            if _small_ok(_small_store(a.data_ptr(), a.stride(0), weight.data_ptr(), y.data_ptr(), y.stride(0),
+                                      int(out_dtype == torch.float32), *_small_tail(a, weight.shape[0], weight)),
+                         "linear_small_m"):
+                return y
         y = gemm(a, weight.t(), out_dtype=out_dtype)
         if y is not NotImplemented:
             return y
@@ -72,6 +120,15 @@ def embed_dyt_cuda(x, tokens, table, alpha, w, b):
 def linear_residual_dyt_cuda(x, a, weight, *rest, mult, has_norm, has_inject):
     norm = rest[:3] if has_norm else None
     tokens, table = rest[-2:] if has_inject else (None, None)
+    if (_small(a, weight) and x.dtype == torch.float32 and x.is_contiguous() and a.shape[0] <= x.shape[0]
+            and (tokens is None or (_i32(tokens) and table.dtype == a.dtype and table.is_contiguous())) and _f32(*(norm or ()))):
+        h = torch.empty((a.shape[0], x.shape[1]), dtype=a.dtype, device=a.device) if has_norm else None
+        alpha, nw, nb = norm or (None, None, None)
+        rc = _small_residual(a.data_ptr(), a.stride(0), weight.data_ptr(), x.data_ptr(), float(mult), _ptr(tokens), _ptr(table),
+                             table.shape[0] if has_inject else 0, _ptr(alpha), _ptr(nw), _ptr(nb), _ptr(h),
+                             *_small_tail(a, weight.shape[0], weight))
+        if _small_ok(rc, "linear_small_m_residual"):
+            return h if has_norm else ()
     y = product(a, weight)
     return stream_dyt(x, y, mult, tokens.reshape(-1) if tokens is not None else None, table, norm, a.dtype)
 
@@ -98,6 +155,11 @@ def linear_rows_cuda(a, weight, out_dtype):
 @native("linear_swiglu")
 def linear_swiglu_cuda(h, weight):
     f = weight.shape[0] // 2
+    if _small(h, weight):
+        y = torch.empty((h.shape[0], f), dtype=h.dtype, device=h.device)
+        if _small_ok(_small_swiglu(h.data_ptr(), h.stride(0), weight.data_ptr(), y.data_ptr(), *_small_tail(h, f, weight)),
+                     "linear_small_m_swiglu"):
+            return y
     gu = product(h, weight)
     y = torch.empty((h.shape[0], f), dtype=h.dtype, device=h.device)
     rc = _swiglu_packed(gu.data_ptr(), y.data_ptr(), h.shape[0], f, _CODE[h.dtype], _stream())
@@ -111,8 +173,13 @@ def min_gru_cuda(h, weight, bz, bx, state, pos, count, T):
     B, width = state.shape
     if not _f32(bz, bx, state) or not _i32(pos, count) or not state.is_contiguous() or h.shape[0] != B * T:
         return NotImplemented
-    zxg = product(h, weight)
     y = torch.empty((B * T, width), dtype=h.dtype, device=h.device)
+    if T == 1 and _small(h, weight):
+        rc = _small_min_gru(h.data_ptr(), h.stride(0), weight.data_ptr(), bz.data_ptr(), bx.data_ptr(), state.data_ptr(),
+                            pos.data_ptr(), count.data_ptr(), y.data_ptr(), *_small_tail(h, width, weight))
+        if _small_ok(rc, "linear_small_m_min_gru"):
+            return y
+    zxg = product(h, weight)
     rc = _min_gru(zxg.data_ptr(), bz.data_ptr(), bx.data_ptr(), state.data_ptr(), y.data_ptr(), pos.data_ptr(),
                   count.data_ptr(), B, T, width, _CODE[h.dtype], _stream())
     if rc == -1:
@@ -132,6 +199,19 @@ def diff_attention_cuda(qkv, cos, sin, kc, vc, pos, count, lam, T, heads, rotary
         return NotImplemented
     code, s = _CODE[qkv.dtype], _stream()
     out = torch.empty((B * T, heads * vdim), dtype=qkv.dtype, device=qkv.device)
+    if T == 1 and qkv.dtype == torch.bfloat16 and dim % 8 == 0 and vdim % 8 == 0 and dim <= 128 and vdim <= 256:
+        units = B * G * ((heads // G + 7) // 8)
+        longest = min(smax, chunk) if chunk else smax
+        splits = max(1, min((2 * _sms(qkv.device) + units - 1) // units, (longest + 63) // 64, 64))
+        counters = _scratch(qkv.device)[2]
+        part = torch.empty(units * splits * 16 * (vdim + 2), dtype=torch.float32, device=qkv.device) if splits > 1 else None
+        if units <= counters.numel():
+            rc = _diff_decode(qkv.data_ptr(), qkv.stride(0), _ptr(cos), _ptr(sin), kc.data_ptr(), vc.data_ptr(), out.data_ptr(),
+                              out.stride(0), pos.data_ptr(), count.data_ptr(), lam.data_ptr(), B, heads, G, dim, vdim,
+                              rotary_dim, smax, chunk, float(scale), float(eps), float(out_scale), splits, _ptr(part),
+                              counters.data_ptr(), s)
+            if _small_ok(rc, "diff_attn_decode"):
+                return out
     rc = _rope_append(qkv.data_ptr(), qkv.stride(0), _ptr(cos), _ptr(sin), kc.data_ptr(), vc.data_ptr(), pos.data_ptr(),
                       count.data_ptr(), B, T, heads, G, dim, vdim, rotary_dim, smax, code, s)
     if rc == -1:
@@ -154,7 +234,3 @@ def advance_by_cuda(pos, count):
     _count("advance_by")
     return pos
 
-
-# kept importable by name for tests that drive one kernel at a time
-__all__ = ["product", "stream_dyt"] + [n for n in list(globals()) if n.endswith("_cuda")]
-assert "diff_attention_" in OPS

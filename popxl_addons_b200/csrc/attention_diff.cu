@@ -69,6 +69,45 @@ __global__ void __launch_bounds__(256)
   }
 }
 
+// The same for sizes that are multiples of eight (dim, vdim, R even): eight features per thread through 16-byte accesses.
+template <typename T> struct alignas(16) Pack16 { T v[16 / sizeof(T)]; };
+template <typename T>
+__global__ void __launch_bounds__(256)
+    diff_rope_append_vec_kernel(T* __restrict__ qkv, long long ld, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
+                                T* __restrict__ kc, T* __restrict__ vc, const int* __restrict__ pos, const int* __restrict__ count,
+                                int T_len, int H, int G, int dim, int vdim, int R, int Smax) {
+  constexpr int V = 16 / sizeof(T);
+  const int b = blockIdx.y, t = blockIdx.x, p = pos[b] + t;
+  if (t >= count[b] || p < 0 || p >= Smax) return;
+  T* src = qkv + ((long long)b * T_len + t) * ld;
+  const float* cs = cos_t + (long long)p * (R / 2);
+  const float* sn = sin_t + (long long)p * (R / 2);
+  const int per = dim / V, nq = H * 2 * per, nk = G * 2 * per, per_v = vdim / V, nv = G * per_v;
+  for (int u = threadIdx.x; u < nq + nk + nv; u += blockDim.x) {
+    if (u < nq + nk) {
+      const bool is_q = u < nq;
+      const int w = is_q ? u : u - nq, hm = w / per, e = (w - hm * per) * V;
+      if (is_q && e >= R) continue;  // passes unchanged, in place
+      T* sp = src + (is_q ? 0 : (long long)H * 2 * dim) + (long long)hm * dim + e;
+      Pack16<T> x = *reinterpret_cast<const Pack16<T>*>(sp);
+#pragma unroll
+      for (int i = 0; i < V; i += 2) {
+        if (e + i < R) {
+          const float c = cs[(e + i) / 2], s = sn[(e + i) / 2], x0 = xl_to_float(x.v[i]), x1 = xl_to_float(x.v[i + 1]);
+          x.v[i] = xl_from_float<T>(x0 * c - x1 * s);
+          x.v[i + 1] = xl_from_float<T>(x1 * c + x0 * s);
+        }
+      }
+      if (is_q) *reinterpret_cast<Pack16<T>*>(sp) = x;
+      else *reinterpret_cast<Pack16<T>*>(kc + (((long long)b * G * 2 + hm) * Smax + p) * dim + e) = x;
+    } else {
+      const int w = u - nq - nk, g = w / per_v, e = (w - g * per_v) * V;
+      *reinterpret_cast<Pack16<T>*>(vc + (((long long)b * G + g) * Smax + p) * vdim + e) =
+          *reinterpret_cast<const Pack16<T>*>(src + (long long)(H + G) * 2 * dim + (long long)g * vdim + e);
+    }
+  }
+}
+
 // ---- general kernel --------------------------------------------------------------------------------------------------
 constexpr int DG_WARPS = 4;
 constexpr int DG_MAX_DIM = 256;   // query / key features per map
@@ -159,7 +198,8 @@ __global__ void __launch_bounds__(DG_WARPS * 32)
 constexpr int DD_WARPS = 4;
 constexpr int DD_KEYS = 16;       // keys per block
 constexpr int DD_HEADS = 8;       // query heads per CTA
-constexpr int DD_RING_LIMIT = 96 * 1024;
+constexpr int DD_RING_LIMIT = 104 * 1024;
+constexpr int DD_MAX_SPLITS = 64;
 
 struct DecodeParams {
   const __nv_bfloat16* qkv;
@@ -201,6 +241,7 @@ __global__ void __launch_bounds__(DD_WARPS * 32) diff_attn_decode_kernel(const D
   extern __shared__ __align__(16) uint8_t smem[];
   __shared__ __align__(16) __nv_bfloat16 sq[2][DD_HEADS][KD * 32];
   __shared__ float sm[DD_WARPS][16], sl[DD_WARPS][16];
+  __shared__ float wt[DD_MAX_SPLITS * 16], wl[DD_MAX_SPLITS * 16];  // maxima, then weights, and sums of the slices
   __shared__ unsigned int is_last;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, quad = lane >> 2, j = lane & 3;
   const int per_g = p.H / p.G, hchunks = (per_g + DD_HEADS - 1) / DD_HEADS;
@@ -217,45 +258,7 @@ __global__ void __launch_bounds__(DD_WARPS * 32) diff_attn_decode_kernel(const D
   const __nv_bfloat16* kb = p.kc + ((long long)b * p.G + g) * 2 * p.Smax * p.dim;
   const __nv_bfloat16* vb = p.vc + ((long long)b * p.G + g) * p.Smax * p.vdim;
 
-  // ---- rotated queries to shared memory; the CTAs with the last keys append the new key and value (the same data each) ----
-  const int half = p.dim / 2;  // dim is even
-  auto rotated = [&](const __nv_bfloat16* s, int e, float& y0, float& y1) {
-    const float x0 = __bfloat162float(s[0]), x1 = __bfloat162float(s[1]);
-    if (e < p.R) {
-      const float c = p.cos_t[(long long)pos * (p.R / 2) + e / 2], sn = p.sin_t[(long long)pos * (p.R / 2) + e / 2];
-      y0 = x0 * c - x1 * sn;
-      y1 = x1 * c + x0 * sn;
-    } else {
-      y0 = x0;
-      y1 = x1;
-    }
-  };
-  for (int i = threadIdx.x; i < 2 * DD_HEADS * KD * 16; i += blockDim.x) {
-    const int e = (i % (KD * 16)) * 2, hm = i / (KD * 16), m = hm / DD_HEADS, r = hm % DD_HEADS;
-    float y0 = 0.f, y1 = 0.f;
-    if (r < nh && e < p.dim) rotated(row + ((long long)(h0 + r) * 2 + m) * p.dim + e, e, y0, y1);
-    *reinterpret_cast<uint32_t*>(&sq[m][r][e]) = dd_pack(y0, y1);
-  }
-  if (split == splits - 1) {
-    for (int i = threadIdx.x; i < 2 * half; i += blockDim.x) {
-      const int m = i / half, e = (i % half) * 2;
-      float y0, y1;
-      rotated(row + ((long long)(p.H + g) * 2 + m) * p.dim + e, e, y0, y1);
-      *reinterpret_cast<uint32_t*>(p.kc + ((((long long)b * p.G + g) * 2 + m) * p.Smax + pos) * p.dim + e) = dd_pack(y0, y1);
-    }
-    const __nv_bfloat16* vsrc = row + (long long)(p.H + p.G) * 2 * p.dim + (long long)g * p.vdim;
-    __nv_bfloat16* vdst = p.vc + (((long long)b * p.G + g) * p.Smax + pos) * p.vdim;
-    for (int i = threadIdx.x; i < p.vdim; i += blockDim.x) vdst[i] = vsrc[i];
-    __threadfence();
-  }
-  __syncthreads();
-  uint4 q1[KD], q2[KD];
-#pragma unroll
-  for (int i = 0; i < KD; ++i) {
-    q1[i] = *reinterpret_cast<const uint4*>(&sq[0][quad][i * 32 + j * 8]);
-    q2[i] = *reinterpret_cast<const uint4*>(&sq[1][quad][i * 32 + j * 8]);
-  }
-  // ---- key blocks ---------------------------------------------------------------------------------------------------------
+  // ---- the ring of key / value blocks: a range without the new key starts to load right away --------------------------------
   const int stage_bytes = dd_stage_bytes(KD, p.vdim), vld = p.vdim + 8;
   uint8_t* ring = smem + (long long)warp * p.stages * stage_bytes;
   const int mine = (blk1 - blk0 - warp + DD_WARPS - 1) / DD_WARPS;  // this warp's blocks: blk0 + warp, + DD_WARPS, ...
@@ -285,6 +288,47 @@ __global__ void __launch_bounds__(DD_WARPS * 32) diff_attn_decode_kernel(const D
     }
     asm volatile("cp.async.commit_group;" ::: "memory");  // possibly empty: keeps the group count per block fixed
   };
+  const bool appends = split == splits - 1;
+  if (!appends)
+    for (int n = 0; n < p.stages - 1; ++n) prefetch(n);
+  // ---- rotated queries to shared memory; the CTAs with the last keys append the new key and value (the same data each) ----
+  const int half = p.dim / 2;  // dim is even
+  auto rotated = [&](const __nv_bfloat16* s, int e, float& y0, float& y1) {
+    const float x0 = __bfloat162float(s[0]), x1 = __bfloat162float(s[1]);
+    if (e < p.R) {
+      const float c = p.cos_t[(long long)pos * (p.R / 2) + e / 2], sn = p.sin_t[(long long)pos * (p.R / 2) + e / 2];
+      y0 = x0 * c - x1 * sn;
+      y1 = x1 * c + x0 * sn;
+    } else {
+      y0 = x0;
+      y1 = x1;
+    }
+  };
+  for (int i = threadIdx.x; i < 2 * DD_HEADS * KD * 16; i += blockDim.x) {
+    const int e = (i % (KD * 16)) * 2, hm = i / (KD * 16), m = hm / DD_HEADS, r = hm % DD_HEADS;
+    float y0 = 0.f, y1 = 0.f;
+    if (r < nh && e < p.dim) rotated(row + ((long long)(h0 + r) * 2 + m) * p.dim + e, e, y0, y1);
+    *reinterpret_cast<uint32_t*>(&sq[m][r][e]) = dd_pack(y0, y1);
+  }
+  if (appends) {
+    for (int i = threadIdx.x; i < 2 * half; i += blockDim.x) {
+      const int m = i / half, e = (i % half) * 2;
+      float y0, y1;
+      rotated(row + ((long long)(p.H + g) * 2 + m) * p.dim + e, e, y0, y1);
+      *reinterpret_cast<uint32_t*>(p.kc + ((((long long)b * p.G + g) * 2 + m) * p.Smax + pos) * p.dim + e) = dd_pack(y0, y1);
+    }
+    const __nv_bfloat16* vsrc = row + (long long)(p.H + p.G) * 2 * p.dim + (long long)g * p.vdim;
+    __nv_bfloat16* vdst = p.vc + (((long long)b * p.G + g) * p.Smax + pos) * p.vdim;
+    for (int i = threadIdx.x; i < p.vdim; i += blockDim.x) vdst[i] = vsrc[i];
+    __threadfence();
+  }
+  __syncthreads();
+  uint4 q1[KD], q2[KD];
+#pragma unroll
+  for (int i = 0; i < KD; ++i) {
+    q1[i] = *reinterpret_cast<const uint4*>(&sq[0][quad][i * 32 + j * 8]);
+    q2[i] = *reinterpret_cast<const uint4*>(&sq[1][quad][i * 32 + j * 8]);
+  }
   float o[VT][4];
 #pragma unroll
   for (int t = 0; t < VT; ++t)
@@ -292,7 +336,8 @@ __global__ void __launch_bounds__(DD_WARPS * 32) diff_attn_decode_kernel(const D
     for (int e = 0; e < 4; ++e) o[t][e] = 0.f;
   float mx[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};  // rows quad (map 1) and quad + 8 (map 2)
   const float sc = p.scale * 1.4426950408889634f;
-  for (int n = 0; n < p.stages - 1; ++n) prefetch(n);
+  if (appends)
+    for (int n = 0; n < p.stages - 1; ++n) prefetch(n);
   for (int n = 0; n < mine; ++n) {
     prefetch(n + p.stages - 1);
     if (p.stages == 2) asm volatile("cp.async.wait_group 1;" ::: "memory");
@@ -413,9 +458,8 @@ __global__ void __launch_bounds__(DD_WARPS * 32) diff_attn_decode_kernel(const D
     }
   }
   __syncthreads();
-  for (int i = threadIdx.x; i < 16 * p.vdim; i += blockDim.x) {
-    const int r = i / p.vdim, c = i % p.vdim;
-    if ((r & 7) >= nh) continue;
+  for (int i = threadIdx.x; i < 2 * nh * p.vdim; i += blockDim.x) {
+    const int rr = i / p.vdim, c = i - rr * p.vdim, r = rr < nh ? rr : DD_HEADS + rr - nh;  // rows in use
     float acc = 0.f;
 #pragma unroll
     for (int w = 0; w < DD_WARPS; ++w)
@@ -431,27 +475,28 @@ __global__ void __launch_bounds__(DD_WARPS * 32) diff_attn_decode_kernel(const D
     if (!is_last) return;
     __threadfence();
     const float* parts = p.part + unit * splits * 16 * pw;
-    if (threadIdx.x < 16) {
-      const int r = threadIdx.x;
-      float m = -INFINITY, ll = 0.f;
-      for (int k = 0; k < splits; ++k) m = fmaxf(m, __ldcg(parts + ((long long)k * 16 + r) * pw));
-      for (int k = 0; k < splits; ++k) {
-        const float mk = __ldcg(parts + ((long long)k * 16 + r) * pw);
-        ll += mk == -INFINITY ? 0.f : __ldcg(parts + ((long long)k * 16 + r) * pw + 1) * exp2f(mk - m);
-      }
-      fm[r] = m;
-      fl[r] = ll;
+    for (int i = threadIdx.x; i < splits * 16; i += blockDim.x) {
+      wt[i] = __ldcg(parts + (long long)i * pw);
+      wl[i] = __ldcg(parts + (long long)i * pw + 1);
     }
     __syncthreads();
-    for (int i = threadIdx.x; i < 16 * p.vdim; i += blockDim.x) {
-      const int r = i / p.vdim, c = i % p.vdim;
-      if ((r & 7) >= nh) continue;
-      float acc = 0.f;
+    if (threadIdx.x < 16) {
+      float m = -INFINITY, ll = 0.f;
+      for (int k = 0; k < splits; ++k) m = fmaxf(m, wt[k * 16 + threadIdx.x]);
       for (int k = 0; k < splits; ++k) {
-        const float* src = parts + ((long long)k * 16 + r) * pw;
-        const float mk = __ldcg(src);
-        if (mk != -INFINITY) acc += __ldcg(src + 2 + c) * exp2f(mk - fm[r]);
+        float& w = wt[k * 16 + threadIdx.x];
+        w = w == -INFINITY ? 0.f : exp2f(w - m);
+        ll += w * wl[k * 16 + threadIdx.x];
       }
+      fl[threadIdx.x] = ll;
+    }
+    __syncthreads();
+    for (int i = threadIdx.x; i < 2 * nh * p.vdim; i += blockDim.x) {
+      const int rr = i / p.vdim, c = i - rr * p.vdim, r = rr < nh ? rr : DD_HEADS + rr - nh;
+      const float* src = parts + (long long)r * pw + 2 + c;
+      float acc = 0.f;
+#pragma unroll 8
+      for (int k = 0; k < splits; ++k) acc += wt[k * 16 + r] * __ldcg(src + (long long)k * 16 * pw);
       so[(long long)r * p.vdim + c] = acc;
     }
     if (threadIdx.x == 0) p.counters[unit] = 0;
@@ -501,6 +546,14 @@ XL_API int xl_diff_rope_append(void* qkv, long long ld, const float* cos_t, cons
   if (R > 0 && (!cos_t || !sin_t)) return -1;
   const long long rows = (long long)B * T_len;
   const long long items = rows * ((long long)(H + G) * 2 * ((dim + 1) / 2) + (long long)G * ((vdim + 1) / 2));
+  if (dim % 8 == 0 && vdim % 8 == 0 && ld % 8 == 0 && B <= 65535 && ((uintptr_t)qkv & 15) == 0 && ((uintptr_t)kc & 15) == 0 &&
+      ((uintptr_t)vc & 15) == 0) {
+    XL_DISPATCH_DTYPE(dtype, T, {
+      diff_rope_append_vec_kernel<T><<<dim3(T_len, B), 256, 0, s>>>((T*)qkv, ld, cos_t, sin_t, (T*)kc, (T*)vc, pos, count, T_len,
+                                                                   H, G, dim, vdim, R, Smax);
+    });
+    return (int)cudaGetLastError();
+  }
   XL_DISPATCH_DTYPE(dtype, T, {
     diff_rope_append_kernel<T><<<xl_grid_for(items, 256), 256, 0, s>>>((T*)qkv, ld, cos_t, sin_t, (T*)kc, (T*)vc, pos, count,
                                                                       rows, T_len, H, G, dim, vdim, R, Smax);
@@ -534,7 +587,7 @@ XL_API int xl_diff_attn_decode(const void* qkv, long long ld, const float* cos_t
                                int dim, int vdim, int R, int Smax, int chunk, float scale, float eps, float out_scale,
                                int splits, float* part, unsigned int* counters, cudaStream_t s) {
   if (B < 1 || B > 65535 || G < 1 || H % G || H > 4096 || dim < 8 || dim > 128 || dim % 8 || vdim < 8 || vdim > 256 || vdim % 8 ||
-      R < 0 || R > dim || (R & 1) || Smax < 1 || chunk < 0 || splits < 1 || splits > 1024 || (ld % 8))
+      R < 0 || R > dim || (R & 1) || Smax < 1 || chunk < 0 || splits < 1 || splits > DD_MAX_SPLITS || (ld % 8))
     return -1;
   if (((uintptr_t)qkv & 15) || ((uintptr_t)kc & 15) || ((uintptr_t)vc & 15) || (R > 0 && (!cos_t || !sin_t))) return -1;
   if (splits > 1 && (!part || !counters)) return -1;

@@ -6,8 +6,8 @@
 //   min_gru    weight rows [z | u | g], one row per sequence: one step of the recurrence on the fp32 state
 //
 // The product is bandwidth-bound (at most 16 multiply-adds per weight), so it uses `mma.sync.m16n8k16` with operands from
-// registers: each lane copies 32 contiguous bytes of a weight row through a per-warp cp.async ring and feeds them to four
-// MMAs. (Any assignment of k indices to the k slots of an MMA is valid as long as both operands agree.)
+// registers: each lane copies two 16-byte pieces of a weight row (four lanes: 64 contiguous bytes each time) through a per-warp
+// cp.async ring and feeds them to four MMAs; the activations it needs for them are loaded one chunk ahead into registers. (Any assignment of k indices to the k slots of an MMA is valid as long as both operands agree.)
 //
 // Work = (column tiles) x (K chunks of 64), tile-major, cut into equal contiguous ranges, one per CTA, so the grid fits the
 // machine and not the problem. A tile shared by several CTAs is finished by the one that arrives last: every CTA leaves its
@@ -22,7 +22,7 @@ namespace {
 
 constexpr int SM_WARPS = 4;
 constexpr int SM_KC = 64;       // k values per chunk (16 per lane)
-constexpr int SM_STAGES = 2;
+constexpr int SM_STAGES = 3;
 constexpr int SM_CTAS_PER_SM = 2;
 
 enum SmMode : int { SM_STORE = 0, SM_RESIDUAL = 1, SM_SWIGLU = 2, SM_MINGRU = 3 };
@@ -32,7 +32,7 @@ template <int MODE> struct SmTile {
   static constexpr int CH = MODE == SM_SWIGLU ? 32 : (MODE == SM_MINGRU ? 16 : 64);  // channels per tile
   static constexpr int COLS = PARTS * CH;
   static constexpr int NT = COLS / 8;
-  static constexpr int STAGE = (NT + 2) * 2 * 32;  // uint4: NT weight pieces and two activation rows, 2 x 16 bytes a lane
+  static constexpr int STAGE = NT * 2 * 32;  // uint4: two pieces of NT weight rows per lane
   static constexpr int RING_BYTES = SM_WARPS * SM_STAGES * STAGE * 16;
 };
 
@@ -107,7 +107,15 @@ __device__ __forceinline__ void sm_epilogue(const SmParams& p, int r, int c, con
   }
 }
 
-__device__ __forceinline__ long long sm_begin(long long total, int cta, int grid) { return total * cta / grid; }
+// Contiguous ranges of items: the first `rem` CTAs take per + 1 items, the others per.
+struct SmRanges {
+  int per, rem;
+  __device__ __forceinline__ int begin(int cta) const { return cta * per + min(cta, rem); }
+  __device__ __forceinline__ int owner(int item) const {
+    const int head = rem * (per + 1);
+    return item < head ? item / (per + 1) : rem + (item - head) / per;
+  }
+};
 
 template <int MODE>
 __global__ void __launch_bounds__(SM_WARPS * 32, SM_CTAS_PER_SM) linear_small_m_kernel(const SmParams p) {
@@ -121,91 +129,98 @@ __global__ void __launch_bounds__(SM_WARPS * 32, SM_CTAS_PER_SM) linear_small_m_
   const int channels = p.N / PARTS;
   const int chunks = (p.K + SM_KC - 1) / SM_KC;
   const int n_tiles = (channels + CH - 1) / CH;
-  const long long total = (long long)n_tiles * chunks;
-  const int grid = (int)gridDim.x;
-  long long item = sm_begin(total, blockIdx.x, grid);
-  const long long item_end = sm_begin(total, blockIdx.x + 1, grid);
-  const int first_tile = (int)(item / chunks);
+  const int total = n_tiles * chunks;
+  const SmRanges ranges{total / (int)gridDim.x, total % (int)gridDim.x};
+  int item = ranges.begin(blockIdx.x);
+  const int item_end = ranges.begin(blockIdx.x + 1);
+  const int first_tile = item / chunks;
   uint4* ring = ring_all + warp * (SM_STAGES * L::STAGE);
 
-  auto prefetch = [&](int tile, int ch, int buf) {
-    const int k0 = ch * SM_KC + j * 16;
-    uint4* dst = ring + buf * L::STAGE + lane;
-#pragma unroll
-    for (int t = 0; t < NT; ++t) {
-      const int col = t * 8 + quad, part = col / CH, c = tile * CH + col % CH;
-      const bool row_on = c < channels;
-      const __nv_bfloat16* src = p.w + ((long long)part * channels + (row_on ? c : 0)) * p.K;
-#pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        const bool on = row_on && k0 + e * 8 < p.K;
-        cp_async16(dst + (t * 2 + e) * 32, src + (on ? k0 + e * 8 : 0), on);
-      }
+  // The chunks of this warp over the whole range, tile after tile: (tile, chunk) of the next one to request and of the next to
+  // multiply advance by the same rule.
+  struct Cursor { int item, c1, ch, tile; };  // first item of the current tile segment, its end chunk, current chunk
+  auto segment = [&](Cursor& c) {  // enter the segment that starts at c.item (or stop at the end of the range)
+    while (c.item < item_end) {
+      c.tile = c.item / chunks;
+      const int c0 = c.item - c.tile * chunks;
+      c.c1 = min(chunks, c0 + (item_end - c.item));
+      c.ch = c0 + warp;
+      if (c.ch < c.c1) return;
+      c.item += c.c1 - c0;
     }
-#pragma unroll
-    for (int hi = 0; hi < 2; ++hi) {
-      const int r = quad + hi * 8;
-#pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        const bool on = r < p.M && k0 + e * 8 < p.K;
-        cp_async16(dst + ((NT + hi) * 2 + e) * 32, p.a + (on ? (long long)r * p.lda + k0 + e * 8 : 0), on);
-      }
-    }
-    asm volatile("cp.async.commit_group;" ::: "memory");
   };
-
+  auto advance = [&](Cursor& c) {
+    c.ch += SM_WARPS;
+    if (c.ch >= c.c1) {
+      c.item = c.tile * chunks + c.c1;
+      segment(c);
+    }
+  };
+  auto request = [&](const Cursor& c, int buf) {
+    if (c.item < item_end) {
+      const int k0 = c.ch * SM_KC + j * 8;
+      uint4* dst = ring + buf * L::STAGE + lane;
+#pragma unroll
+      for (int t = 0; t < NT; ++t) {
+        const int col = t * 8 + quad, part = col / CH, n = c.tile * CH + col % CH;
+        const bool row_on = n < channels;
+        const __nv_bfloat16* src = p.w + ((long long)part * channels + (row_on ? n : 0)) * p.K;
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const bool on = row_on && k0 + e * 32 < p.K;
+          cp_async16(dst + (t * 2 + e) * 32, src + (on ? k0 + e * 32 : 0), on);
+        }
+      }
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");  // possibly empty: one group per chunk slot
+  };
+  auto load_a = [&](const Cursor& c, uint4 (&lo)[2], uint4 (&hi)[2]) {
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int k = c.ch * SM_KC + j * 8 + e * 32;
+      const bool on = c.item < item_end && k < p.K;
+      lo[e] = on && quad < p.M ? *reinterpret_cast<const uint4*>(p.a + (long long)quad * p.lda + k) : make_uint4(0, 0, 0, 0);
+      hi[e] = on && quad + 8 < p.M ? *reinterpret_cast<const uint4*>(p.a + (long long)(quad + 8) * p.lda + k) : make_uint4(0, 0, 0, 0);
+    }
+  };
+  Cursor ahead{item, 0, 0, 0};
+  segment(ahead);
+  Cursor cur = ahead;
+  uint4 a_lo[2], a_hi[2];
+  load_a(cur, a_lo, a_hi);
+#pragma unroll
+  for (int n = 0; n < SM_STAGES - 1; ++n) {
+    request(ahead, n);
+    if (ahead.item < item_end) advance(ahead);
+  }
   int buf = 0;
-  bool have = false;  // ring[buf] holds (or is receiving) this warp's first chunk of the current tile
   while (item < item_end) {
-    const int tile = (int)(item / chunks);
-    const int c0 = (int)(item - (long long)tile * chunks);
-    const int c1 = (int)min((long long)chunks, c0 + (item_end - item));
+    const int tile = item / chunks;
+    const int c0 = item - tile * chunks;
+    const int c1 = min(chunks, c0 + (item_end - item));
     float acc[NT][4];
 #pragma unroll
     for (int t = 0; t < NT; ++t)
 #pragma unroll
       for (int e = 0; e < 4; ++e) acc[t][e] = 0.f;
-    if (!have && c0 + warp < c1) prefetch(tile, c0 + warp, buf);
-    have = false;
     for (int ch = c0 + warp; ch < c1; ch += SM_WARPS) {
-      // request the chunk after this one: the next of this tile, or this warp's first of the next tile
-      bool next = false;
-      if (ch + SM_WARPS < c1) {
-        prefetch(tile, ch + SM_WARPS, buf ^ 1);
-        next = true;
-      } else {
-        const long long nit = item + (c1 - c0);
-        if (nit < item_end) {
-          const int nc1 = (int)min((long long)chunks, item_end - nit);  // the next tile starts at its first chunk
-          if (warp < nc1) {
-            prefetch(tile + 1, warp, buf ^ 1);
-            next = have = true;
-          }
-        }
-      }
-      if (next) asm volatile("cp.async.wait_group 1;" ::: "memory");
-      else asm volatile("cp.async.wait_group 0;" ::: "memory");
+      request(ahead, (buf + SM_STAGES - 1) % SM_STAGES);
+      if (ahead.item < item_end) advance(ahead);
+      uint4 lo[2] = {a_lo[0], a_lo[1]}, hi[2] = {a_hi[0], a_hi[1]};
+      advance(cur);
+      load_a(cur, a_lo, a_hi);
+      asm volatile("cp.async.wait_group %0;" ::"n"(SM_STAGES - 1) : "memory");
       const uint4* src = ring + buf * L::STAGE + lane;  // every lane reads back the pieces it copied itself
-      buf ^= 1;
-      uint32_t lo[8], hi[8];
-#pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        *reinterpret_cast<uint4*>(lo + 4 * e) = src[(NT * 2 + e) * 32];
-        *reinterpret_cast<uint4*>(hi + 4 * e) = src[((NT + 1) * 2 + e) * 32];
-      }
+      buf = (buf + 1) % SM_STAGES;
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         uint4 w[NT];
 #pragma unroll
         for (int t = 0; t < NT; ++t) w[t] = src[(t * 2 + e) * 32];
 #pragma unroll
-        for (int s = 0; s < 2; ++s)
+        for (int t = 0; t < NT; ++t) mma_bf16(acc[t], lo[e].x, hi[e].x, lo[e].y, hi[e].y, w[t].x, w[t].y);
 #pragma unroll
-          for (int t = 0; t < NT; ++t) {
-            const uint32_t* ww = reinterpret_cast<const uint32_t*>(&w[t]);
-            mma_bf16(acc[t], lo[4 * e + 2 * s], hi[4 * e + 2 * s], lo[4 * e + 2 * s + 1], hi[4 * e + 2 * s + 1], ww[2 * s],
-                     ww[2 * s + 1]);
-          }
+        for (int t = 0; t < NT; ++t) mma_bf16(acc[t], lo[e].z, hi[e].z, lo[e].w, hi[e].w, w[t].z, w[t].w);
       }
     }
     __syncthreads();  // readers of the previous tile are done with `red`
@@ -237,15 +252,13 @@ __global__ void __launch_bounds__(SM_WARPS * 32, SM_CTAS_PER_SM) linear_small_m_
       if (finishing) __threadfence();
     }
     if (finishing) {
-      // CTAs that share the tile, in order
-      int cta0 = blockIdx.x, cta1 = blockIdx.x;
+      // CTAs that share the tile, in order. All but the first begin inside it: it is their first tile (slot 0). It is the
+      // last tile of the first one, and its first only if that one begins exactly with it.
+      int cta0 = blockIdx.x, cta1 = blockIdx.x, slot0 = 0;
       if (!whole) {
-        const long long lo_item = (long long)tile * chunks, hi_item = lo_item + chunks - 1;
-        cta0 = (int)(lo_item * grid / total);
-        while (cta0 > 0 && sm_begin(total, cta0, grid) > lo_item) --cta0;
-        while (sm_begin(total, cta0 + 1, grid) <= lo_item) ++cta0;
-        cta1 = cta0;
-        while (sm_begin(total, cta1 + 1, grid) <= hi_item) ++cta1;
+        cta0 = ranges.owner(tile * chunks);
+        cta1 = ranges.owner(tile * chunks + chunks - 1);
+        slot0 = ranges.begin(cta0) < tile * chunks ? 1 : 0;
       }
       for (int i = threadIdx.x; i < p.M * CH; i += blockDim.x) {
         const int r = i / CH, cc = i % CH, c = tile * CH + cc;
@@ -259,10 +272,9 @@ __global__ void __launch_bounds__(SM_WARPS * 32, SM_CTAS_PER_SM) linear_small_m_
 #pragma unroll
             for (int w = 0; w < SM_WARPS; ++w) s += red[w][r][col];
           } else {
-            for (int k = cta0; k <= cta1; ++k) {
-              const int which = (int)(sm_begin(total, k, grid) / chunks) == tile ? 0 : 1;
-              s += __ldcg(p.slots + ((long long)k * 2 + which) * (16 * COLS) + r * COLS + col);
-            }
+            s = __ldcg(p.slots + ((long long)cta0 * 2 + slot0) * (16 * COLS) + r * COLS + col);
+#pragma unroll 4
+            for (int k = cta0 + 1; k <= cta1; ++k) s += __ldcg(p.slots + (long long)k * 2 * (16 * COLS) + r * COLS + col);
           }
           v[q] = s;
         }
@@ -288,6 +300,7 @@ template <int MODE> int sm_launch(const SmParams& p, int sms, int max_tiles, cud
   }
   long long grid = (long long)SM_CTAS_PER_SM * sms;
   const long long total = (long long)n_tiles * chunks;
+  if (total > (1 << 30)) return -1;
   if (grid > total) grid = total;
   linear_small_m_kernel<MODE><<<(int)grid, SM_WARPS * 32, L::RING_BYTES, s>>>(p);
   return (int)cudaGetLastError();

@@ -9,10 +9,7 @@
 // Rows of a portion are (sequence, token) with `T` tokens per sequence; `count[b]` of them are real, the rest is padding.
 #include "common.cuh"
 
-#include <cooperative_groups.h>
 #include <math.h>
-
-namespace cg = cooperative_groups;
 
 namespace {
 
@@ -124,136 +121,130 @@ __global__ void advance_by_kernel(int* pos, const int* count, int n) {
 // ------------------------------------------------------------------------------------------------------------------
 // minGRU over a portion. zxg: (B*T, 3W) rows [z | candidate | output gate] pre-activations without biases. Every channel
 // is an independent first-order recurrence, and composing steps is associative: (a, b) then (a', b') = (a a', a' b + b').
-// A CTA owns 32*V channels and 16 warps x 8 tokens; a cluster of CTAs covers consecutive token ranges of the same channels
-// and exchanges the range totals through distributed shared memory, so all operands are read from memory exactly once.
-// The state (B, W) stays in fp32; a sequence at position 0 starts from zero whatever the state buffer holds.
+// The portion is cut into ranges of `L` tokens. The first kernel composes every range but the last to one (a, b) per channel;
+// in the second, each range folds its predecessors' pairs onto the state it starts from and walks its tokens. A portion of
+// one range needs only the second. One thread per range and V channels; loads of GRU_AHEAD tokens are in flight together.
+// The state (B, W) stays in fp32; a sequence at position 0 starts from zero whatever the state buffer holds. All ranges read
+// the old state, so the new one waits in the last slot of `pairs` until a third, tiny kernel stores it.
 // ------------------------------------------------------------------------------------------------------------------
-constexpr int GRU_WARPS = 16;
-constexpr int GRU_STEPS = 8;
-constexpr int GRU_TILE = GRU_WARPS * GRU_STEPS;  // tokens per CTA and iteration
-constexpr int GRU_MAX_CLUSTER = 8;
+constexpr int GRU_THREADS = 128;
+constexpr int GRU_AHEAD = 8;
+constexpr int GRU_MAX_RANGES = 64;
+
+// 32-bit models: the correctly rounded forms; 16-bit models: the same functions by the hardware's exponential and division
+template <typename T> __device__ __forceinline__ float gate_sigmoid(float x) { return __fdividef(1.f, 1.f + __expf(-x)); }
+template <> __device__ __forceinline__ float gate_sigmoid<float>(float x) { return sigmoid_f(x); }
+
+struct GruParams {
+  const float *bz, *bx;
+  float* state;
+  float2* pairs;  // [B][ranges][W]
+  const int *pos, *count;
+  int T, W, L, ranges;
+};
 
 template <typename T, int V>
-__global__ void __launch_bounds__(GRU_WARPS * 32)
-    min_gru_kernel(const T* __restrict__ zxg, const float* __restrict__ bz, const float* __restrict__ bx,
-                   float* __restrict__ state, T* __restrict__ y, const int* __restrict__ pos, const int* __restrict__ count,
-                   int T_len, int W) {
-  __shared__ float2 part[GRU_WARPS][32 * V];
-  __shared__ float2 total[2][32 * V];  // double-buffered: a CTA of the cluster may still read the previous iteration's
-  cg::cluster_group cluster = cg::this_cluster();
-  const int C = (int)cluster.num_blocks(), rank = (int)cluster.block_rank();
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  const int b = blockIdx.z;
-  const int ch = (blockIdx.y * 32 + lane) * V;
-  const bool on = ch < W;  // W is a multiple of V
-  const int cnt = min(count[b], T_len);
-  float bzv[V], bxv[V], carry[V];
+__device__ __forceinline__ void gru_step(const float (&zr)[V], const float (&ur)[V], const float (&bz)[V], const float (&bx)[V],
+                                         float (&a)[V], float (&b)[V]) {
 #pragma unroll
   for (int e = 0; e < V; ++e) {
-    bzv[e] = on ? bz[ch + e] : 0.f;
-    bxv[e] = on ? bx[ch + e] : 0.f;
-    carry[e] = (on && pos[b] > 0) ? state[(long long)b * W + ch + e] : 0.f;
+    const float z = gate_sigmoid<T>(zr[e] + bz[e]), u = ur[e] + bx[e];
+    a[e] = 1.f - z;
+    b[e] = z * (u >= 0.f ? u + 0.5f : gate_sigmoid<T>(u));
   }
-  int buf = 0;
-  for (int t0 = 0; t0 < cnt; t0 += C * GRU_TILE, buf ^= 1) {
-    const int t_first = t0 + rank * GRU_TILE + warp * GRU_STEPS;
-    float a[GRU_STEPS][V], bb[GRU_STEPS][V], g[GRU_STEPS][V];
+}
+
+template <typename T, int V, bool OUTPUT>
+__global__ void __launch_bounds__(GRU_THREADS) min_gru_kernel(const T* __restrict__ zxg, T* __restrict__ y, const GruParams p) {
+  const int ch = (blockIdx.x * GRU_THREADS + threadIdx.x) * V;
+  const int range = blockIdx.y, b = blockIdx.z;
+  const int cnt = min(p.count[b], p.T);
+  const int t0 = range * p.L, t1 = min(cnt, t0 + p.L);
+  if (ch >= p.W || t0 >= t1) return;
+  const long long W = p.W;
+  float bz[V], bx[V], S[V], A[V];
+  load_pack<float, V>(p.bz + ch, bz);
+  load_pack<float, V>(p.bx + ch, bx);
 #pragma unroll
-    for (int s = 0; s < GRU_STEPS; ++s) {
-      if (on && t_first + s < cnt) {
-        const T* row = zxg + ((long long)b * T_len + t_first + s) * 3 * W + ch;
-        load_pack<T, V>(row, a[s]);
-        load_pack<T, V>(row + W, bb[s]);
-        load_pack<T, V>(row + 2 * W, g[s]);
-      } else {
+  for (int e = 0; e < V; ++e) { S[e] = 0.f; A[e] = 1.f; }
+  if (OUTPUT) {
+    if (p.pos[b] > 0) load_pack<float, V>(p.state + b * W + ch, S);
+    const float2* src = p.pairs + (long long)b * p.ranges * W + ch;
+#pragma unroll 4
+    for (int r = 0; r < range; ++r) {
+      float ab[2 * V];
+      load_pack<float, 2 * V>(reinterpret_cast<const float*>(src + r * W), ab);
 #pragma unroll
-        for (int e = 0; e < V; ++e) a[s][e] = bb[s][e] = g[s][e] = 0.f;
-      }
+      for (int e = 0; e < V; ++e) S[e] = ab[2 * e] * S[e] + ab[2 * e + 1];
     }
-    float A[V], B[V];
+  }
+  const T* row = zxg + ((long long)b * p.T + t0) * 3 * W + ch;
+  T* out = OUTPUT ? y + ((long long)b * p.T + t0) * W + ch : nullptr;
+  for (int t = t0; t < t1; t += GRU_AHEAD) {
+    float z[GRU_AHEAD][V], u[GRU_AHEAD][V], g[GRU_AHEAD][V];
 #pragma unroll
-    for (int e = 0; e < V; ++e) { A[e] = 1.f; B[e] = 0.f; }
-#pragma unroll
-    for (int s = 0; s < GRU_STEPS; ++s) {
-      const bool real = t_first + s < cnt;
-#pragma unroll
-      for (int e = 0; e < V; ++e) {
-        const float z = sigmoid_f(a[s][e] + bzv[e]);
-        const float u = bb[s][e] + bxv[e];
-        const float c = u >= 0.f ? u + 0.5f : sigmoid_f(u);
-        a[s][e] = real ? 1.f - z : 1.f;
-        bb[s][e] = real ? z * c : 0.f;
-        B[e] = a[s][e] * B[e] + bb[s][e];
-        A[e] *= a[s][e];
-      }
+    for (int i = 0; i < GRU_AHEAD; ++i) {
+      const T* src = row + (long long)(t - t0 + (t + i < t1 ? i : 0)) * 3 * W;
+      load_pack<T, V>(src, z[i]);
+      load_pack<T, V>(src + W, u[i]);
+      if (OUTPUT) load_pack<T, V>(src + 2 * W, g[i]);
     }
 #pragma unroll
-    for (int e = 0; e < V; ++e) part[warp][lane * V + e] = make_float2(A[e], B[e]);
-    __syncthreads();
-    if (warp == GRU_WARPS - 1) {
+    for (int i = 0; i < GRU_AHEAD; ++i) {
+      if (t + i < t1) {
+        float a[V], c[V];
+        gru_step<T, V>(z[i], u[i], bz, bx, a, c);
 #pragma unroll
-      for (int e = 0; e < V; ++e) {
-        float2 acc = make_float2(1.f, 0.f);
-        for (int w = 0; w < GRU_WARPS; ++w) {
-          const float2 p = part[w][lane * V + e];
-          acc = make_float2(acc.x * p.x, p.x * acc.y + p.y);
+        for (int e = 0; e < V; ++e) {
+          S[e] = a[e] * S[e] + c[e];
+          A[e] *= a[e];
         }
-        total[buf][lane * V + e] = acc;
+        if (OUTPUT) {
+          float o[V];
+#pragma unroll
+          for (int e = 0; e < V; ++e) o[e] = S[e] * g[i][e] * gate_sigmoid<T>(g[i][e]);
+          store_pack<T, V>(out + (long long)(t - t0 + i) * W, o);
+        }
       }
     }
-    cluster.sync();
-    float S[V];
-#pragma unroll
-    for (int e = 0; e < V; ++e) {
-      S[e] = carry[e];
-      for (int r = 0; r < C; ++r) {
-        const float2 p = cluster.map_shared_rank(&total[buf][0], r)[lane * V + e];
-        if (r == rank) S[e] = carry[e];
-        carry[e] = p.x * carry[e] + p.y;
-      }
-      for (int w = 0; w < warp; ++w) {
-        const float2 p = part[w][lane * V + e];
-        S[e] = p.x * S[e] + p.y;
-      }
-    }
-#pragma unroll
-    for (int s = 0; s < GRU_STEPS; ++s) {
-      float o[V];
-#pragma unroll
-      for (int e = 0; e < V; ++e) {
-        S[e] = a[s][e] * S[e] + bb[s][e];
-        o[e] = S[e] * silu_f(g[s][e]);
-      }
-      if (on && t_first + s < cnt) store_pack<T, V>(y + ((long long)b * T_len + t_first + s) * W + ch, o);
-    }
-    __syncthreads();  // `part` is rewritten by the next iteration
   }
-  if (rank == 0 && warp == 0 && on) {
+  if (OUTPUT) {
+    // the state at the end of the portion, after the last pair of this sequence (ranges of other CTAs still read `state`)
+    if (t1 == cnt) {
+      float s2[2 * V];
 #pragma unroll
-    for (int e = 0; e < V; ++e) state[(long long)b * W + ch + e] = carry[e];
+      for (int e = 0; e < V; ++e) { s2[2 * e] = 0.f; s2[2 * e + 1] = S[e]; }
+      store_pack<float, 2 * V>(reinterpret_cast<float*>(p.pairs + ((long long)b * p.ranges + p.ranges - 1) * W + ch), s2);
+    }
+  } else {
+    float ab[2 * V];
+#pragma unroll
+    for (int e = 0; e < V; ++e) { ab[2 * e] = A[e]; ab[2 * e + 1] = S[e]; }
+    store_pack<float, 2 * V>(reinterpret_cast<float*>(p.pairs + ((long long)b * p.ranges + range) * W + ch), ab);
   }
-  cluster.sync();  // no CTA leaves while another may still read its totals
+}
+
+__global__ void __launch_bounds__(256) min_gru_commit_kernel(const GruParams p) {
+  const int c = blockIdx.x * blockDim.x + threadIdx.x, b = blockIdx.y;
+  if (c < p.W && min(p.count[b], p.T) > 0)
+    p.state[(long long)b * p.W + c] = p.pairs[((long long)b * p.ranges + p.ranges - 1) * p.W + c].y;
+}
+
+inline int gru_range(int T) {
+  int L = (T + GRU_MAX_RANGES - 2) / (GRU_MAX_RANGES - 1);  // one slot of `pairs` is left for the final state
+  L = (L + GRU_AHEAD - 1) / GRU_AHEAD * GRU_AHEAD;
+  return L < 32 ? 32 : L;
 }
 
 template <typename T, int V>
-int launch_min_gru(const void* zxg, const float* bz, const float* bx, float* state, void* y, const int* pos, const int* count,
-                   int B, int T_len, int W, cudaStream_t s) {
-  const int groups = (W + 32 * V - 1) / (32 * V);
-  int C = 1;
-  while (C < GRU_MAX_CLUSTER && C * GRU_TILE < T_len && (long long)groups * B * C < 2 * 148) C *= 2;
-  cudaLaunchConfig_t cfg = {};
-  cfg.gridDim = dim3(C, groups, B);
-  cfg.blockDim = dim3(GRU_WARPS * 32);
-  cfg.stream = s;
-  cudaLaunchAttribute attr[1];
-  attr[0].id = cudaLaunchAttributeClusterDimension;
-  attr[0].val.clusterDim.x = C;
-  attr[0].val.clusterDim.y = 1;
-  attr[0].val.clusterDim.z = 1;
-  cfg.attrs = attr;
-  cfg.numAttrs = 1;
-  const cudaError_t e = cudaLaunchKernelEx(&cfg, min_gru_kernel<T, V>, (const T*)zxg, bz, bx, state, (T*)y, pos, count, T_len, W);
-  return e != cudaSuccess ? (int)e : (int)cudaGetLastError();
+int launch_min_gru(const void* zxg, void* y, GruParams p, int B, cudaStream_t s) {
+  const int used = (p.T + p.L - 1) / p.L;
+  const dim3 block(GRU_THREADS);
+  const int gx = (p.W + V * GRU_THREADS - 1) / (V * GRU_THREADS);
+  if (used > 1) min_gru_kernel<T, V, false><<<dim3(gx, used - 1, B), block, 0, s>>>((const T*)zxg, (T*)y, p);
+  min_gru_kernel<T, V, true><<<dim3(gx, used, B), block, 0, s>>>((const T*)zxg, (T*)y, p);
+  min_gru_commit_kernel<<<dim3((p.W + 255) / 256, B), 256, 0, s>>>(p);
+  return (int)cudaGetLastError();
 }
 
 template <typename T>
@@ -310,13 +301,22 @@ XL_API int xl_advance_by(int* pos, const int* count, int n, cudaStream_t s) {
   return (int)cudaGetLastError();
 }
 
-// zxg (B*T_len, 3W) and y (B*T_len, W) of type `dtype`; bz, bx (W), state (B, W) fp32; pos, count (B) int32.
-XL_API int xl_min_gru(const void* zxg, const float* bz, const float* bx, float* state, void* y, const int* pos, const int* count,
-                      int B, int T_len, int W, int dtype, cudaStream_t s) {
-  if (B < 1 || B > 65535 || T_len < 1 || W < 1 || (W + 31) / 32 > 65535) return -1;
+// Floats of `pairs` that a portion needs.
+XL_API long long xl_min_gru_scratch(int B, int T_len, int W) {
+  return 2LL * B * ((T_len + gru_range(T_len) - 1) / gru_range(T_len) + 1) * W;
+}
+
+// zxg (B*T_len, 3W) and y (B*T_len, W) of type `dtype`; bz, bx (W), state (B, W), pairs (scratch) fp32; pos, count (B) int32.
+// All base pointers 16-byte aligned. Rows of y past count[b] are not written.
+XL_API int xl_min_gru(const void* zxg, const float* bz, const float* bx, float* state, void* y, float* pairs, const int* pos,
+                      const int* count, int B, int T_len, int W, int dtype, cudaStream_t s) {
+  if (B < 1 || B > 65535 || T_len < 1 || W < 1 || !pairs) return -1;
+  GruParams p;
+  p.bz = bz; p.bx = bx; p.state = state; p.pairs = (float2*)pairs; p.pos = pos; p.count = count; p.T = T_len; p.W = W;
+  p.L = gru_range(T_len);
+  p.ranges = (T_len + p.L - 1) / p.L + 1;
   XL_DISPATCH_DTYPE(dtype, T, {
-    return W % 2 == 0 ? launch_min_gru<T, 2>(zxg, bz, bx, state, y, pos, count, B, T_len, W, s)
-                      : launch_min_gru<T, 1>(zxg, bz, bx, state, y, pos, count, B, T_len, W, s);
+    return W % 2 == 0 ? launch_min_gru<T, 2>(zxg, y, p, B, s) : launch_min_gru<T, 1>(zxg, y, p, B, s);
   });
   return (int)cudaGetLastError();
 }

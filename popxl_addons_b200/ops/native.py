@@ -212,7 +212,13 @@ def check_gemm_errors():
                      21: "CTA-pair GEMM: operand tiles never arrived (TMA)",
                      22: "CTA-pair GEMM: shared-memory stage was never released",
                      23: "CTA-pair GEMM: accumulator never completed",
-                     24: "CTA-pair GEMM: accumulator buffer was never drained"}
+                     24: "CTA-pair GEMM: accumulator buffer was never drained",
+                     41: "differential attention: query tiles never arrived",
+                     42: "differential attention: key / value tile never arrived",
+                     43: "differential attention: key / value stage was never released",
+                     44: "differential attention: scores never completed",
+                     45: "differential attention: probabilities never arrived",
+                     46: "differential attention: output accumulation never completed"}
             raise RuntimeError(f"tcgen05 GEMM on cuda:{idx} gave up waiting: {names.get(code, code)}")
 
 

@@ -3,19 +3,23 @@
 import torch
 
 from ..xl.opdef import native
-from .native import (_CODE, _c_f, _c_int, _c_ll, _c_p, _check, _count, _ok, _sig, _sms, _stream, gemm)
+from .native import (_CODE, _c_f, _c_int, _c_ll, _c_p, _check, _count, _ok, _sig, _sms, _stream, gemm,
+                     gemm_error_flag)
 
 _stream_dyt = _sig("xl_stream_dyt", _c_p, _c_p, _c_f, _c_p, _c_p, _c_int, _c_p, _c_p, _c_p, _c_p, _c_ll, _c_int, _c_int, _c_p)
 _select_dyt = _sig("xl_select_dyt", _c_p, _c_p, _c_int, _c_int, _c_ll, _c_p, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int, _c_p)
 _swiglu_packed = _sig("xl_swiglu_packed", _c_p, _c_p, _c_ll, _c_int, _c_int, _c_p)
 _advance_by = _sig("xl_advance_by", _c_p, _c_p, _c_int, _c_p)
-_min_gru = _sig("xl_min_gru", _c_p, _c_p, _c_p, _c_p, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int, _c_p)
+_min_gru = _sig("xl_min_gru", _c_p, _c_p, _c_p, _c_p, _c_p, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int, _c_p)
+_min_gru_scratch = _sig("xl_min_gru_scratch", _c_int, _c_int, _c_int, restype=_c_ll)
 _rope_append = _sig("xl_diff_rope_append", _c_p, _c_ll, _c_p, _c_p, _c_p, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int,
                     _c_int, _c_int, _c_int, _c_int, _c_int, _c_p)
 _diff_general = _sig("xl_diff_attn_general", _c_p, _c_ll, _c_p, _c_p, _c_p, _c_ll, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int,
                      _c_int, _c_int, _c_int, _c_int, _c_int, _c_f, _c_f, _c_f, _c_int, _c_p)
 _diff_decode = _sig("xl_diff_attn_decode", _c_p, _c_ll, _c_p, _c_p, _c_p, _c_p, _c_p, _c_ll, _c_p, _c_p, _c_p, _c_int, _c_int,
                     _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_f, _c_f, _c_f, _c_int, _c_p, _c_p, _c_p)
+_diff_tcgen05 = _sig("xl_diff_attn_tcgen05", _c_p, _c_ll, _c_p, _c_p, _c_p, _c_ll, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int,
+                     _c_int, _c_int, _c_int, _c_int, _c_f, _c_f, _c_f, _c_p, _c_p)
 _small_m_slots = _sig("xl_linear_small_m_slots", _c_int)
 _SMALL_TAIL = (_c_int, _c_int, _c_int, _c_p, _c_p, _c_int, _c_int, _c_p)
 _small_store = _sig("xl_linear_small_m", _c_p, _c_ll, _c_p, _c_p, _c_ll, _c_int, *_SMALL_TAIL)
@@ -180,7 +184,8 @@ def min_gru_cuda(h, weight, bz, bx, state, pos, count, T):
         if _small_ok(rc, "linear_small_m_min_gru"):
             return y
     zxg = product(h, weight)
-    rc = _min_gru(zxg.data_ptr(), bz.data_ptr(), bx.data_ptr(), state.data_ptr(), y.data_ptr(), pos.data_ptr(),
+    pairs = torch.empty(_min_gru_scratch(B, T, width), dtype=torch.float32, device=h.device)
+    rc = _min_gru(zxg.data_ptr(), bz.data_ptr(), bx.data_ptr(), state.data_ptr(), y.data_ptr(), pairs.data_ptr(), pos.data_ptr(),
                   count.data_ptr(), B, T, width, _CODE[h.dtype], _stream())
     if rc == -1:
         return NotImplemented
@@ -202,7 +207,7 @@ def diff_attention_cuda(qkv, cos, sin, kc, vc, pos, count, lam, T, heads, rotary
     if T == 1 and qkv.dtype == torch.bfloat16 and dim % 8 == 0 and vdim % 8 == 0 and dim <= 128 and vdim <= 256:
         units = B * G * ((heads // G + 7) // 8)
         longest = min(smax, chunk) if chunk else smax
-        splits = max(1, min((2 * _sms(qkv.device) + units - 1) // units, (longest + 63) // 64, 64))
+        splits = max(1, min(2 * _sms(qkv.device) // units, (longest + 63) // 64, 64))  # one wave, two CTAs per SM
         counters = _scratch(qkv.device)[2]
         part = torch.empty(units * splits * 16 * (vdim + 2), dtype=torch.float32, device=qkv.device) if splits > 1 else None
         if units <= counters.numel():
@@ -218,6 +223,14 @@ def diff_attention_cuda(qkv, cos, sin, kc, vc, pos, count, lam, T, heads, rotary
         return NotImplemented
     _check(rc, "diff_rope_append")
     _count("diff_rope_append")
+    if qkv.dtype == torch.bfloat16:
+        rc = _diff_tcgen05(qkv.data_ptr(), qkv.stride(0), kc.data_ptr(), vc.data_ptr(), out.data_ptr(), out.stride(0),
+                           pos.data_ptr(), count.data_ptr(), lam.data_ptr(), B, T, heads, G, dim, vdim, smax, chunk, float(scale),
+                           float(eps), float(out_scale), gemm_error_flag(qkv.device).data_ptr(), s)
+        if rc >= 0:
+            _check(rc, "diff_attn_tcgen05")
+            _count("diff_attn_tcgen05")
+            return out
     rc = _diff_general(qkv.data_ptr(), qkv.stride(0), kc.data_ptr(), vc.data_ptr(), out.data_ptr(), out.stride(0),
                        pos.data_ptr(), count.data_ptr(), lam.data_ptr(), B, T, heads, G, dim, vdim, smax, chunk, float(scale),
                        float(eps), float(out_scale), code, s)

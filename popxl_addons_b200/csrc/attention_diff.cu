@@ -110,10 +110,9 @@ __global__ void __launch_bounds__(256)
 
 // ---- general kernel --------------------------------------------------------------------------------------------------
 constexpr int DG_WARPS = 4;
-constexpr int DG_MAX_DIM = 256;   // query / key features per map
-constexpr int DG_VPL = 8;         // value features per lane: vdim <= 256
+constexpr int DG_MAX_DIM = 512;   // query / key features per map; value features: 32 per DG_VPL, at most 512
 
-template <typename T>
+template <typename T, int DG_VPL>
 __global__ void __launch_bounds__(DG_WARPS * 32)
     diff_attn_general_kernel(const T* __restrict__ q, long long ldq, const T* __restrict__ kc, const T* __restrict__ vc,
                              T* __restrict__ out, long long ldo, const int* __restrict__ pos, const int* __restrict__ count,
@@ -249,7 +248,10 @@ __global__ void __launch_bounds__(DD_WARPS * 32) diff_attn_decode_kernel(const D
   const int h0 = g * per_g + (blockIdx.y % hchunks) * DD_HEADS;  // first query head of this CTA
   const int nh = min(DD_HEADS, (g + 1) * per_g - h0);
   const int pos = p.pos[b];
-  if (p.count[b] <= 0 || pos < 0 || pos >= p.Smax) return;
+  if (p.count[b] <= 0 || pos < 0 || pos >= p.Smax) {
+    xl_grid_dependency_wait();  // no kernel of a chain ends before its predecessor
+    return;
+  }
   const int first = p.chunk > 0 ? (pos / p.chunk) * p.chunk : 0;
   const int len = pos + 1 - first;
   const int blocks = (len + DD_KEYS - 1) / DD_KEYS;
@@ -291,6 +293,8 @@ __global__ void __launch_bounds__(DD_WARPS * 32) diff_attn_decode_kernel(const D
   const bool appends = split == splits - 1;
   if (!appends)
     for (int n = 0; n < p.stages - 1; ++n) prefetch(n);
+  xl_grid_dependency_wait();  // the new projections; positions and older keys were there before the previous kernel started
+  xl_grid_launch_dependents();
   // ---- rotated queries to shared memory; the CTAs with the last keys append the new key and value (the same data each) ----
   const int half = p.dim / 2;  // dim is even
   auto rotated = [&](const __nv_bfloat16* s, int e, float& y0, float& y1) {
@@ -532,8 +536,9 @@ template <int KD, int VT> int dd_launch(DecodeParams p, int B, int splits, cudaS
     configured = bytes;
   }
   const int hchunks = (p.H / p.G + DD_HEADS - 1) / DD_HEADS;
-  diff_attn_decode_kernel<KD, VT><<<dim3(splits, p.G * hchunks, B), DD_WARPS * 32, bytes, s>>>(p);
-  return (int)cudaGetLastError();
+  const cudaError_t e = xl_launch_overlapped(diff_attn_decode_kernel<KD, VT>, dim3(splits, p.G * hchunks, B), dim3(DD_WARPS * 32),
+                                             (size_t)bytes, s, p);
+  return e != cudaSuccess ? (int)e : (int)cudaGetLastError();
 }
 
 }  // namespace
@@ -561,20 +566,25 @@ XL_API int xl_diff_rope_append(void* qkv, long long ld, const float* cos_t, cons
   return (int)cudaGetLastError();
 }
 
-// q: (B*T_len, ldq), rotated; out: (B*T_len, ldo). dim <= 256, vdim <= 256. chunk 0: plain causal. Rows past count[b] of a
+// q: (B*T_len, ldq), rotated; out: (B*T_len, ldo). dim <= 512, vdim <= 512. chunk 0: plain causal. Rows past count[b] of a
 // sequence are left as they are.
 XL_API int xl_diff_attn_general(const void* q, long long ldq, const void* kc, const void* vc, void* out, long long ldo,
                                 const int* pos, const int* count, const float* lam, int B, int T_len, int H, int G, int dim,
                                 int vdim, int Smax, int chunk, float scale, float eps, float out_scale, int dtype,
                                 cudaStream_t s) {
   if (B < 1 || B > 65535 || H < 1 || H > 65535 || T_len < 1 || G < 1 || H % G || dim < 1 || dim > DG_MAX_DIM || vdim < 1 ||
-      vdim > 32 * DG_VPL || Smax < 1 || chunk < 0)
+      vdim > 512 || Smax < 1 || chunk < 0)
     return -1;
   const dim3 grid((T_len + DG_WARPS - 1) / DG_WARPS, H, B);
   XL_DISPATCH_DTYPE(dtype, T, {
-    diff_attn_general_kernel<T><<<grid, DG_WARPS * 32, 0, s>>>((const T*)q, ldq, (const T*)kc, (const T*)vc, (T*)out, ldo, pos,
-                                                              count, lam, T_len, H, G, dim, vdim, Smax, chunk, scale, eps,
-                                                              out_scale);
+    if (vdim <= 256)
+      diff_attn_general_kernel<T, 8><<<grid, DG_WARPS * 32, 0, s>>>((const T*)q, ldq, (const T*)kc, (const T*)vc, (T*)out, ldo,
+                                                                   pos, count, lam, T_len, H, G, dim, vdim, Smax, chunk, scale,
+                                                                   eps, out_scale);
+    else
+      diff_attn_general_kernel<T, 16><<<grid, DG_WARPS * 32, 0, s>>>((const T*)q, ldq, (const T*)kc, (const T*)vc, (T*)out, ldo,
+                                                                    pos, count, lam, T_len, H, G, dim, vdim, Smax, chunk, scale,
+                                                                    eps, out_scale);
   });
   return (int)cudaGetLastError();
 }

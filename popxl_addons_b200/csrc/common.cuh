@@ -87,3 +87,25 @@ static inline int xl_grid_for(long long n_items, int per_block, int max_blocks =
   if (b > max_blocks) b = max_blocks;
   return (int)b;
 }
+
+// Programmatic dependent launch: the kernel may start while its predecessor on the stream drains. It must call
+// xl_grid_dependency_wait() before it touches anything the predecessor reads or writes; what it does before (loading weights,
+// which nothing in flight writes) overlaps the predecessor's tail. xl_grid_launch_dependents() after that wait lets the
+// successor do the same, so at most two kernels of a chain are in flight. Both are no-ops in an ordinary launch.
+__device__ __forceinline__ void xl_grid_dependency_wait() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
+__device__ __forceinline__ void xl_grid_launch_dependents() { asm volatile("griddepcontrol.launch_dependents;" ::: "memory"); }
+
+template <typename... P, typename... A>
+static inline cudaError_t xl_launch_overlapped(void (*kernel)(P...), dim3 grid, dim3 block, size_t smem, cudaStream_t s, A... args) {
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = grid;
+  cfg.blockDim = block;
+  cfg.dynamicSmemBytes = smem;
+  cfg.stream = s;
+  cudaLaunchAttribute attr[1];
+  attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  attr[0].val.programmaticStreamSerializationAllowed = 1;
+  cfg.attrs = attr;
+  cfg.numAttrs = 1;
+  return cudaLaunchKernelEx(&cfg, kernel, args...);
+}

@@ -12,7 +12,7 @@
 // Work = (column tiles) x (K chunks of 64), tile-major, cut into equal contiguous ranges, one per CTA, so the grid fits the
 // machine and not the problem. A tile shared by several CTAs is finished by the one that arrives last: every CTA leaves its
 // partial sums in a slot of its own and the finisher adds the slots in CTA order, so results do not depend on timing.
-// Nobody waits for anybody. An epilogue that combines several weight rows per output channel (swiglu, min_gru) takes them
+// No CTA waits for another. Consecutive kernels overlap: a launch requests its first weights while its predecessor drains. An epilogue that combines several weight rows per output channel (swiglu, min_gru) takes them
 // into one tile: a tile is PARTS groups of CH channels, group p starting at weight row p * N / PARTS.
 #include "common.cuh"
 
@@ -186,13 +186,15 @@ __global__ void __launch_bounds__(SM_WARPS * 32, SM_CTAS_PER_SM) linear_small_m_
   Cursor ahead{item, 0, 0, 0};
   segment(ahead);
   Cursor cur = ahead;
-  uint4 a_lo[2], a_hi[2];
-  load_a(cur, a_lo, a_hi);
 #pragma unroll
   for (int n = 0; n < SM_STAGES - 1; ++n) {
     request(ahead, n);
     if (ahead.item < item_end) advance(ahead);
   }
+  xl_grid_dependency_wait();  // the first weights are on their way; everything else may come from the previous kernel
+  xl_grid_launch_dependents();
+  uint4 a_lo[2], a_hi[2];
+  load_a(cur, a_lo, a_hi);
   int buf = 0;
   while (item < item_end) {
     const int tile = item / chunks;
@@ -302,8 +304,9 @@ template <int MODE> int sm_launch(const SmParams& p, int sms, int max_tiles, cud
   const long long total = (long long)n_tiles * chunks;
   if (total > (1 << 30)) return -1;
   if (grid > total) grid = total;
-  linear_small_m_kernel<MODE><<<(int)grid, SM_WARPS * 32, L::RING_BYTES, s>>>(p);
-  return (int)cudaGetLastError();
+  const cudaError_t e = xl_launch_overlapped(linear_small_m_kernel<MODE>, dim3((unsigned)grid), dim3(SM_WARPS * 32),
+                                             L::RING_BYTES, s, p);
+  return e != cudaSuccess ? (int)e : (int)cudaGetLastError();
 }
 
 int sm_check(const void* a, long long lda, const void* w, int M, int N, int K, const float* slots, const unsigned int* counters) {

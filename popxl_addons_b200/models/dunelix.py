@@ -22,8 +22,9 @@ __all__ = ["DunelixConfig", "LayerConfig", "MinGRUConfig", "DiffAttentionConfig"
 
 
 def _take(d: Mapping[str, Any], where: str, required: Tuple[str, ...], optional: Tuple[str, ...] = ()) -> Dict[str, Any]:
-    """The entries of a configuration object; an entry this design does not have is an error, not something to ignore."""
-    unknown = set(d) - set(required) - set(optional)
+    """The entries of a configuration object; an entry this design does not have is an error, not something to ignore (unless
+    it is there only to say that something is absent)."""
+    unknown = {k for k, v in d.items() if v is not None and v is not False} - set(required) - set(optional)
     missing = set(required) - set(d)
     if unknown or missing:
         raise ValueError(f"{where}: unknown entries {sorted(unknown)}, missing entries {sorted(missing)}")
@@ -79,6 +80,8 @@ class LayerConfig:
             mixer = DiffAttentionConfig(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), float(m["diff"]),
                                         float(m["scale"]), int(mask["size"]),
                                         RotaryConfig.from_dict(m["rot"]) if m["rot"] else None)
+            if max(mixer.dim, mixer.vdim) > 512:
+                raise ValueError(f"the attention kernels take dim and vdim up to 512, not {mixer.dim} and {mixer.vdim}")
             if mixer.heads % mixer.kv_heads:
                 raise ValueError(f"heads ({mixer.heads}) must be a multiple of kv_heads ({mixer.kv_heads})")
             if mixer.rot and (mixer.rot.dims % 2 or mixer.rot.dims > mixer.dim):

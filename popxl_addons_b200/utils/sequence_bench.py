@@ -137,7 +137,7 @@ def decode_rows(b, nat, ns, C=4096, F=11008, M=16):
         b.row(f"diff_attn_decode B={B} H={H} G={G} 2x{d}/{dv} len={n}", lambda: (randn(B, G, 2, smax, d), randn(B, G, smax, dv)),
               lambda kc, vc: ns.diff_attention_cuda(q, cos, cos, kc, vc, pos, cnt, lam, 1, H, d, 0, d ** -0.5, 1e-6, 0.4),
               B * G * n * (2 * d + dv) * 2)
-    for B, H, D, n in ((16, 16, 128, 576), (16, 8, 128, 2048)):
+    for B, H, D, n in ((16, 16, 128, 576), (16, 8, 128, 2048), (1, 8, 128, 8192)):
         qkv, p = randn(B, 3 * H * D), torch.tensor(n - 1, dtype=torch.int32, device="cuda")
         b.row(f"  like: attn_decode B={B} H={H} D={D} len={n}", lambda: (randn(B, H, n + 64, D), randn(B, H, n + 64, D)),
               lambda kc, vc: nat.attention_decode_packed_cuda(qkv, kc, vc, p, H, D, D ** -0.5), 2 * B * H * n * D * 2)

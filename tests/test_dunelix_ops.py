@@ -159,6 +159,8 @@ SHAPES = [  # H, G, dim, vdim, rot, chunk, positions
     (2, 1, 40, 72, 12, 64, 200),
     (4, 1, 128, 128, 64, 256, 520),
     (2, 1, 64, 64, 20, 128, 260),
+    (1, 1, 288, 320, 36, 20, 70),   # beyond what the tensor-core kernels take
+    (2, 1, 16, 16, 2, 1, 40),       # chunks of one position
 ]
 
 

@@ -277,10 +277,10 @@ def run_serving(args):
             continue
         gru = {"type": "mingru", "mixer": {"width": R}, "mlp": {"ff": F, "kind": "dense"}}
         att = {"type": "attention", "mlp": {"ff": F, "kind": "dense"},
-               "mixer": {"heads": H, "kv_heads": G, "dim": 64, "vdim": 128, "diff": 0.6, "scale": 0.125, "mask": {"size": 8192},
+               "mixer": {"heads": H, "kv_heads": G, "dim": 64, "vdim": 128, "diff": 0.5, "scale": 0.125, "mask": {"size": 8192},
                          "rot": {"base": 500000.0, "dims": 64,
-                                 "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}}
-        cfg = DunelixConfig.from_dict({"vocab": vocab, "width": C, "norm": {"eps": 1e-6}, "residual_mult": 0.7,
+                                 "scaling": {"factor": 16.0, "low": 1.0, "high": 4.0, "original": 4096}}}}
+        cfg = DunelixConfig.from_dict({"vocab": vocab, "width": C, "norm": {"eps": 1e-6}, "residual_mult": 0.5,
                                        "layers": [gru, gru, att, gru]})
         model = Dunelix(cfg)
         gen = SequenceGenerator(model, batch=B, max_seq=P + N, max_portion=P, max_new_tokens=N, device="cuda",

@@ -49,7 +49,7 @@ def test_prompt_portions_and_decoding(case, backend):
 
 def test_long_prompt_and_long_decoding(backend):
     """Several blocks of every kernel: hundreds of positions, chunks longer than a tile, then a long decoded tail."""
-    cfg = C.config([C.layer({"width": 72}, 64), C.layer(C.attention(heads=4, kv_heads=2, dim=32, vdim=64, size=150, dims=16), 64),
+    cfg = C.config([C.layer({"width": 72}, 64), C.layer(C.attention(heads=6, kv_heads=2, dim=48, vdim=64, size=150, dims=20), 64),
                     C.layer(C.attention(heads=2, kv_heads=1, dim=64, vdim=128, size=0, dims=64), 0)], width=64, loop=(0, 2, 2))
     ckpt, tokens = C.checkpoint(cfg, 3), C.prompt(cfg, 420)
     want = C.oracle_logits(cfg, ckpt, tokens)

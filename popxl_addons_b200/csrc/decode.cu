@@ -673,6 +673,7 @@ __global__ void __launch_bounds__(256)
   const long long row = blockIdx.x;
   float best = -INFINITY;
   int bi = 0;
+#pragma unroll 8
   for (int i = threadIdx.x; i < valid; i += blockDim.x) {
     const float v = xl_to_float(logits[row * V + i]);
     if (v > best) { best = v; bi = i; }

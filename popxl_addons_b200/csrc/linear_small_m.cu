@@ -77,33 +77,66 @@ __device__ __forceinline__ void mma_bf16(float (&c)[4], uint32_t a0, uint32_t a1
 __device__ __forceinline__ float sigmoid_f(float v) { return 1.f / (1.f + expf(-v)); }
 __device__ __forceinline__ float silu_f(float v) { return v / (1.f + expf(-v)); }
 
+// Four channels c .. c + 3 of row r (those below `channels`). All loads come before the first store: their latencies overlap.
 template <int MODE>
-__device__ __forceinline__ void sm_epilogue(const SmParams& p, int r, int c, const float (&v)[SmTile<MODE>::PARTS], int channels) {
+__device__ __forceinline__ void sm_epilogue(const SmParams& p, int r, int c, const float (&v)[SmTile<MODE>::PARTS][4], int channels) {
+  constexpr int LAST = SmTile<MODE>::PARTS - 1;
+  const int n = min(4, channels - c);
+  const long long at = (long long)r * channels + c, yat = (long long)r * p.ldy + c;
   if (MODE == SM_STORE) {
-    if (p.y_f32) ((float*)p.y)[(long long)r * p.ldy + c] = v[0];
-    else ((__nv_bfloat16*)p.y)[(long long)r * p.ldy + c] = __float2bfloat16_rn(v[0]);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      if (e < n) {
+        if (p.y_f32) ((float*)p.y)[yat + e] = v[0][e];
+        else ((__nv_bfloat16*)p.y)[yat + e] = __float2bfloat16_rn(v[0][e]);
+      }
+    }
   } else if (MODE == SM_RESIDUAL) {
-    float* xp = p.x + (long long)r * channels + c;
-    float s = *xp + p.mult * v[0];
-    if (p.table) {
-      const int t = min(max(p.tokens[r], 0), p.vocab - 1);
-      s += __bfloat162float(p.table[(long long)t * channels + c]);
+    float x[4], add[4], nw[4], nb[4];
+    const __nv_bfloat16* row = p.table ? p.table + (long long)min(max(p.tokens[r], 0), p.vocab - 1) * channels + c : nullptr;
+    const float alpha = p.alpha ? *p.alpha : 0.f;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int k = e < n ? e : 0;
+      x[e] = p.x[at + k];
+      add[e] = row ? __bfloat162float(row[k]) : 0.f;
+      nw[e] = p.alpha ? p.nw[c + k] : 0.f;
+      nb[e] = p.alpha ? p.nb[c + k] : 0.f;
     }
-    *xp = s;
-    if (p.alpha) p.h[(long long)r * channels + c] = __float2bfloat16_rn(tanhf(*p.alpha * s) * p.nw[c] + p.nb[c]);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      if (e < n) {
+        const float s = x[e] + p.mult * v[0][e] + add[e];
+        p.x[at + e] = s;
+        if (p.alpha) p.h[at + e] = __float2bfloat16_rn(tanhf(alpha * s) * nw[e] + nb[e]);
+      }
+    }
   } else if (MODE == SM_SWIGLU) {
-    ((__nv_bfloat16*)p.y)[(long long)r * p.ldy + c] = __float2bfloat16_rn(silu_f(v[0]) * v[SmTile<MODE>::PARTS - 1]);
+#pragma unroll
+    for (int e = 0; e < 4; ++e)
+      if (e < n) ((__nv_bfloat16*)p.y)[yat + e] = __float2bfloat16_rn(silu_f(v[0][e]) * v[LAST][e]);
   } else {
-    const float z = sigmoid_f(v[0] + p.bz[c]);
-    const float u = v[1 % SmTile<MODE>::PARTS] + p.bu[c];
-    const float cand = u >= 0.f ? u + 0.5f : sigmoid_f(u);
-    float* sp = p.state + (long long)r * channels + c;
-    float s = p.pos[r] > 0 ? *sp : 0.f;
-    if (p.count[r] > 0) {
-      s = (1.f - z) * s + z * cand;
-      *sp = s;
+    float old[4], bz[4], bu[4];
+    const bool fresh = p.pos[r] <= 0, real = p.count[r] > 0;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int k = e < n ? e : 0;
+      old[e] = fresh ? 0.f : p.state[at + k];
+      bz[e] = p.bz[c + k];
+      bu[e] = p.bu[c + k];
     }
-    ((__nv_bfloat16*)p.y)[(long long)r * p.ldy + c] = __float2bfloat16_rn(s * silu_f(v[SmTile<MODE>::PARTS - 1]));
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      if (e < n) {
+        const float z = sigmoid_f(v[0][e] + bz[e]), u = v[1 % SmTile<MODE>::PARTS][e] + bu[e];
+        float s = old[e];
+        if (real) {
+          s = (1.f - z) * s + z * (u >= 0.f ? u + 0.5f : sigmoid_f(u));
+          p.state[at + e] = s;
+        }
+        ((__nv_bfloat16*)p.y)[yat + e] = __float2bfloat16_rn(s * silu_f(v[LAST][e]));
+      }
+    }
   }
 }
 
@@ -262,23 +295,30 @@ __global__ void __launch_bounds__(SM_WARPS * 32, SM_CTAS_PER_SM) linear_small_m_
         cta1 = ranges.owner(tile * chunks + chunks - 1);
         slot0 = ranges.begin(cta0) < tile * chunks ? 1 : 0;
       }
-      for (int i = threadIdx.x; i < p.M * CH; i += blockDim.x) {
-        const int r = i / CH, cc = i % CH, c = tile * CH + cc;
+      for (int i = threadIdx.x; i < p.M * (CH / 4); i += blockDim.x) {
+        const int r = i / (CH / 4), cc = (i % (CH / 4)) * 4, c = tile * CH + cc;
         if (c >= channels) continue;
-        float v[PARTS];
+        float v[PARTS][4];
 #pragma unroll
         for (int q = 0; q < PARTS; ++q) {
           const int col = q * CH + cc;
-          float s = 0.f;
           if (whole) {
 #pragma unroll
-            for (int w = 0; w < SM_WARPS; ++w) s += red[w][r][col];
+            for (int e = 0; e < 4; ++e) {
+              v[q][e] = 0.f;
+#pragma unroll
+              for (int w = 0; w < SM_WARPS; ++w) v[q][e] += red[w][r][col + e];
+            }
           } else {
-            s = __ldcg(p.slots + ((long long)cta0 * 2 + slot0) * (16 * COLS) + r * COLS + col);
-#pragma unroll 4
-            for (int k = cta0 + 1; k <= cta1; ++k) s += __ldcg(p.slots + (long long)k * 2 * (16 * COLS) + r * COLS + col);
+            const float* base = p.slots + r * COLS + col;
+            float4 t = __ldcg(reinterpret_cast<const float4*>(base + ((long long)cta0 * 2 + slot0) * (16 * COLS)));
+#pragma unroll 8
+            for (int k = cta0 + 1; k <= cta1; ++k) {
+              const float4 o = __ldcg(reinterpret_cast<const float4*>(base + (long long)k * 2 * (16 * COLS)));
+              t.x += o.x; t.y += o.y; t.z += o.z; t.w += o.w;
+            }
+            v[q][0] = t.x; v[q][1] = t.y; v[q][2] = t.z; v[q][3] = t.w;
           }
-          v[q] = s;
         }
         sm_epilogue<MODE>(p, r, c, v, channels);
       }

@@ -1,16 +1,16 @@
 """Model families: GPT-2, GPT-J and Llama shaped decoders assembled from the add-on layers, their training program
-(`DecoderTrainer`) and the int4 tensor-parallel decoding program (`DecoderGenerator`); Dunelix, served from a checkpoint
-folder by `SequenceGenerator`; the registry of architectures (`load_model`)."""
+(`DecoderTrainer`) and the int4 tensor-parallel decoding program (`DecoderGenerator`); Dunelix and Zirunex, served from
+a checkpoint folder by `SequenceGenerator`; the registry of architectures (`load_model`)."""
 from .decoder import DecoderBlock, DecoderConfig, DecoderEmbedding, DecoderHead
 
 __all__ = ["DecoderConfig", "DecoderBlock", "DecoderEmbedding", "DecoderHead", "DecoderTrainer", "PipelineTrainer",
-           "DecoderGenerator", "Dunelix", "DunelixConfig", "SequenceGenerator", "load_model", "load_config",
-           "register_architecture", "ARCHITECTURES"]
+           "DecoderGenerator", "Dunelix", "DunelixConfig", "Zirunex", "ZirunexConfig", "SequenceGenerator", "load_model",
+           "load_config", "register_architecture", "ARCHITECTURES"]
 
 _LAZY = {"DecoderTrainer": "trainer", "PipelineTrainer": "pipeline_trainer", "DecoderGenerator": "generator",
-         "Dunelix": "dunelix", "DunelixConfig": "dunelix", "SequenceGenerator": "sequence_generator",
-         "load_model": "registry", "load_config": "registry", "register_architecture": "registry",
-         "ARCHITECTURES": "registry"}
+         "Dunelix": "dunelix", "DunelixConfig": "dunelix", "Zirunex": "zirunex", "ZirunexConfig": "zirunex",
+         "SequenceGenerator": "sequence_generator", "load_model": "registry", "load_config": "registry",
+         "register_architecture": "registry", "ARCHITECTURES": "registry"}
 
 
 def __getattr__(name):

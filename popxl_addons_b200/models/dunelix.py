@@ -17,18 +17,9 @@ import torch
 from .. import xl
 from ..ops.rotary_pos_embed import frequency_tables, rotary_frequencies
 from ..xl import ops
+from .checkpoint import check_tensors, take
 
 __all__ = ["DunelixConfig", "LayerConfig", "MinGRUConfig", "DiffAttentionConfig", "RotaryConfig", "Dunelix"]
-
-
-def _take(d: Mapping[str, Any], where: str, required: Tuple[str, ...], optional: Tuple[str, ...] = ()) -> Dict[str, Any]:
-    """The entries of a configuration object; an entry this design does not have is an error, not something to ignore (unless
-    it is there only to say that something is absent)."""
-    unknown = {k for k, v in d.items() if v is not None and v is not False} - set(required) - set(optional)
-    missing = set(required) - set(d)
-    if unknown or missing:
-        raise ValueError(f"{where}: unknown entries {sorted(unknown)}, missing entries {sorted(missing)}")
-    return {k: d.get(k) for k in (*required, *optional)}
 
 
 @dataclass(frozen=True)
@@ -39,10 +30,10 @@ class RotaryConfig:
 
     @classmethod
     def from_dict(cls, d):
-        d = _take(d, "rot", ("base", "dims"), ("scaling",))
+        d = take(d, "rot", ("base", "dims"), ("scaling",))
         sc = d["scaling"]
         if sc:
-            sc = tuple(sorted(_take(sc, "rot.scaling", ("factor", "low", "high", "original")).items()))
+            sc = tuple(sorted(take(sc, "rot.scaling", ("factor", "low", "high", "original")).items()))
         return cls(int(d["dims"]), float(d["base"]), sc or None)
 
 
@@ -70,13 +61,13 @@ class LayerConfig:
 
     @classmethod
     def from_dict(cls, d):
-        d = _take(d, "layer", ("type", "mixer"), ("mlp",))
+        d = take(d, "layer", ("type", "mixer"), ("mlp",))
         kind, m = d["type"], d["mixer"]
         if kind == "mingru":
-            mixer = MinGRUConfig(int(_take(m, "mingru", ("width",))["width"]))
+            mixer = MinGRUConfig(int(take(m, "mingru", ("width",))["width"]))
         elif kind == "attention":
-            m = _take(m, "attention", ("heads", "kv_heads", "dim", "vdim", "diff", "scale"), ("mask", "rot"))
-            mask = _take(m["mask"], "mask", ("size",)) if m["mask"] else {"size": 0}
+            m = take(m, "attention", ("heads", "kv_heads", "dim", "vdim", "diff", "scale"), ("mask", "rot"))
+            mask = take(m["mask"], "mask", ("size",)) if m["mask"] else {"size": 0}
             mixer = DiffAttentionConfig(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), float(m["diff"]),
                                         float(m["scale"]), int(mask["size"]),
                                         RotaryConfig.from_dict(m["rot"]) if m["rot"] else None)
@@ -90,7 +81,7 @@ class LayerConfig:
             raise ValueError(f"unknown layer type {kind!r}")
         ff = 0
         if d["mlp"]:
-            mlp = _take(d["mlp"], "mlp", ("ff",), ("kind",))
+            mlp = take(d["mlp"], "mlp", ("ff",), ("kind",))
             if mlp["kind"] not in (None, "dense"):
                 raise ValueError(f"unknown feed-forward kind {mlp['kind']!r}")
             ff = int(mlp["ff"])
@@ -110,16 +101,16 @@ class DunelixConfig:
 
     @classmethod
     def from_dict(cls, d: Mapping[str, Any]) -> "DunelixConfig":
-        d = _take(d, "configuration", ("vocab", "width", "layers", "norm"), ("architecture", "loop", "residual_mult"))
+        d = take(d, "configuration", ("vocab", "width", "layers", "norm"), ("architecture", "loop", "residual_mult"))
         loop = None
         if d["loop"]:
-            lp = _take(d["loop"], "loop", ("start", "stop", "times"))
+            lp = take(d["loop"], "loop", ("start", "stop", "times"))
             loop = (int(lp["start"]), int(lp["stop"]), int(lp["times"]))
             if not 0 <= loop[0] < loop[1] <= len(d["layers"]) or loop[2] < 1:
                 raise ValueError(f"loop {loop} does not fit {len(d['layers'])} layers")
         mult = d["residual_mult"]
         return cls(int(d["vocab"]), int(d["width"]), tuple(LayerConfig.from_dict(e) for e in d["layers"]), loop,
-                   float(_take(d["norm"], "norm", ("eps",))["eps"]), 1.0 if mult is None else float(mult))
+                   float(take(d["norm"], "norm", ("eps",))["eps"]), 1.0 if mult is None else float(mult))
 
     def schedule(self) -> List[Tuple[int, bool]]:
         """Layer runs in order: `(layer, whether the embedding output is added to the stream before it)`."""
@@ -201,13 +192,7 @@ class Dunelix:
 
     def convert(self, ckpt: Mapping[str, torch.Tensor], device) -> Dict[str, torch.Tensor]:
         """Checkpoint tensors -> program tensors (in the checkpoint's precision; the caller casts on copy)."""
-        want = self.checkpoint_tensors()
-        missing, extra = sorted(set(want) - set(ckpt)), sorted(set(ckpt) - set(want))
-        if missing or extra:
-            raise ValueError(f"checkpoint does not fit the configuration: missing {missing[:8]}, unexpected {extra[:8]}")
-        for k, shape in want.items():
-            if tuple(ckpt[k].shape) != shape:
-                raise ValueError(f"checkpoint tensor {k!r} has shape {tuple(ckpt[k].shape)}, expected {shape}")
+        check_tensors(ckpt, self.checkpoint_tensors())
 
         def get(k):
             return ckpt[k].to(device)

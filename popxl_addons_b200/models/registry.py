@@ -39,18 +39,23 @@ def _decoder(family: str):
     return make
 
 
-def _dunelix_config(d: Dict[str, Any]):
-    return import_module(f"{__package__}.dunelix").DunelixConfig.from_dict(d)
+def _served(name: str, module: str) -> Architecture:
+    """An architecture whose module (loaded on first use) has a class `<name>`, which describes the model to
+    `SequenceGenerator`, and its configuration `<name>Config`."""
+    def config(d: Dict[str, Any]):
+        return getattr(import_module(f"{__package__}.{module}"), f"{name}Config").from_dict(d)
 
+    def model(cfg, dtype: str = "bfloat16"):
+        return getattr(import_module(f"{__package__}.{module}"), name)(cfg, dtype)
 
-def _dunelix_model(cfg, dtype: str = "bfloat16"):
-    return import_module(f"{__package__}.dunelix").Dunelix(cfg, dtype)
+    return Architecture(name, config, model)
 
 
 # trained / generated with DecoderTrainer and DecoderGenerator, which take the configuration object
 for _family, _name in (("gptj", "GPT-J"), ("gpt2", "GPT-2"), ("llama", "Llama")):
     register_architecture(Architecture(_name, _decoder(_family)))
-register_architecture(Architecture("Dunelix", _dunelix_config, _dunelix_model))
+for _name, _module in (("Dunelix", "dunelix"), ("Zirunex", "zirunex")):
+    register_architecture(_served(_name, _module))
 
 
 def load_config(folder: str):

@@ -1398,7 +1398,8 @@ from .decode import (rotary_kv_append_, attention_decode_packed, argmax_rows, ad
                      kv_cache_fill_, timestamp, attention_decode_into_, add_layer_norm_,
                      all_reduce_add_layer_norm_)
 from .sequence import (embed_dyt_, linear_residual_dyt_, select_dyt, linear_rows, linear_swiglu, min_gru_,  # noqa: E402
-                       diff_attention_, advance_by_)
+                       diff_attention_, advance_by_, embed_rms_, linear_residual_rms_, select_rms, linear_split_glu,
+                       window_attention_)
 from .extra import *  # noqa: E402,F401,F403
 # module paths of popxl (`ops.call`, `ops.utils`): loaded here so that a later `from ...ops.call import CallSiteInfo`
 # finds the submodule already imported and the name `call` stays bound to the function

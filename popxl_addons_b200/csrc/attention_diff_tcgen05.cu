@@ -269,19 +269,7 @@ __global__ void __launch_bounds__(NUM_THREADS, 1)
           tmem_st_32x32b_x32(tmem_o + ch * 32, raw);
         }
       }
-#pragma unroll
-      for (int ch = 0; ch < BKV / 32; ++ch) {
-        uint32_t hi[16], err[16];
-#pragma unroll
-        for (int i = 0; i < 16; ++i) {
-          const float x = s[ch * 32 + 2 * i], y = s[ch * 32 + 2 * i + 1];
-          asm("cvt.rn.bf16x2.f32 %0, %1, %2;" : "=r"(hi[i]) : "f"(y), "f"(x));
-          const float ex = x - __uint_as_float(hi[i] << 16), ey = y - __uint_as_float(hi[i] & 0xffff0000u);
-          asm("cvt.rn.bf16x2.f32 %0, %1, %2;" : "=r"(err[i]) : "f"(ey), "f"(ex));
-        }
-        tmem_st_32x32b_x16(tmem_s + ch * 16, hi);
-        tmem_st_32x32b_x16(tmem_s + BKV / 2 + ch * 16, err);
-      }
+      store_split_weights<BKV>(tmem_s, s);
       tmem_st_wait();
       tcgen05_fence_before();
       __syncwarp();
@@ -345,29 +333,15 @@ __global__ void __launch_bounds__(NUM_THREADS, 1)
   }
 }
 
-// 2-D map over a row-major bf16 matrix, boxes of {64, box_rows}, 128-byte swizzle
-int make_map(CUtensorMap* map, const void* ptr, long long rows, long long cols, long long ld, int box_rows) {
-  EncodeTiledFn fn = get_encode_fn();
-  if (!fn) return -2;
-  cuuint64_t dims[2] = {(cuuint64_t)cols, (cuuint64_t)rows};
-  cuuint64_t strides[1] = {(cuuint64_t)ld * 2};
-  cuuint32_t box[2] = {64, (cuuint32_t)box_rows};
-  cuuint32_t estr[2] = {1, 1};
-  const CUresult r = fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (void*)ptr, dims, strides, box, estr,
-                        CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
-                        CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
-  return r == CUDA_SUCCESS ? 0 : -3;
-}
-
 template <int DK, int VD>
 int launch(const void* q, long long ldq, const void* kc, const void* vc, const DiffParams& p, int B, cudaStream_t s) {
   using L = DiffSmem<DK, VD>;
   CUtensorMap mq, mk, mv;
-  int r = make_map(&mq, q, (long long)B * p.T, ldq, ldq, BLOCK_Q);
+  int r = make_map_bf16(&mq, q, (long long)B * p.T, ldq, ldq, BLOCK_Q);
   if (r) return r;
-  r = make_map(&mk, kc, (long long)B * p.G * 2 * p.Smax, p.dim, p.dim, BKV);
+  r = make_map_bf16(&mk, kc, (long long)B * p.G * 2 * p.Smax, p.dim, p.dim, BKV);
   if (r) return r;
-  r = make_map(&mv, vc, (long long)B * p.G * p.Smax, p.vdim, p.vdim, 64);
+  r = make_map_bf16(&mv, vc, (long long)B * p.G * p.Smax, p.vdim, p.vdim, 64);
   if (r) return r;
   static bool configured = false;
   if (!configured) {

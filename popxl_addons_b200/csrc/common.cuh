@@ -73,6 +73,12 @@ __device__ __forceinline__ float xl_block_max(float v, float* smem) {
   return xl_warp_max(r);
 }
 
+// Gated unit with clamped inputs: g * sigmoid(slope g) * (u + shift) with g = min(gate, limit), u = clamp(up, -limit, limit).
+__device__ __forceinline__ float xl_clamped_glu_value(float gate, float up, float limit, float slope, float shift) {
+  const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
+  return g / (1.f + expf(-slope * g)) * (u + shift);
+}
+
 #define XL_DISPATCH_DTYPE(dtype, T, ...)                                     \
   switch (dtype) {                                                           \
     case XL_F32: { using T = float; __VA_ARGS__; break; }                    \

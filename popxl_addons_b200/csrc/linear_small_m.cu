@@ -1,9 +1,14 @@
 // Linear layers of the decoding path, bf16 weights, M <= 16 rows: C[M, N] = a[M, K] * w[N, K]^T, the weights streamed once.
 // What follows the product in a layer happens in the epilogue, on the fp32 sums:
 //   store      C as bf16 or fp32
-//   residual   x += mult * C (+ table[token]) on the fp32 residual stream, h = DyT(x) for the next layer
+//   residual   x += mult * C (+ table[token]) on the fp32 residual stream; for the next layer h = DyT(x), or the first half of
+//              an RMS norm: h = x * w and the sums of squares of x over blocks of 64 columns (one column tile each)
 //   swiglu     weight rows [gate | up]: y = silu(gate) * up
+//   split_glu  weight rows [plain | gate | up]: plain results stored, a clamped gated unit of the others beside them
 //   min_gru    weight rows [z | u | g], one row per sequence: one step of the recurrence on the fp32 state
+//
+// store and split_glu may take rows of such a half-done norm: their results are multiplied by 1 / sqrt(mean(x^2) + eps), summed
+// up from the blocks' sums of squares while the weights arrive.
 //
 // The product is bandwidth-bound (at most 16 multiply-adds per weight), so it uses `mma.sync.m16n8k16` with operands from
 // registers: each lane copies two 16-byte pieces of a weight row (four lanes: 64 contiguous bytes each time) through a per-warp
@@ -25,11 +30,12 @@ constexpr int SM_KC = 64;       // k values per chunk (16 per lane)
 constexpr int SM_STAGES = 3;
 constexpr int SM_CTAS_PER_SM = 2;
 
-enum SmMode : int { SM_STORE = 0, SM_RESIDUAL = 1, SM_SWIGLU = 2, SM_MINGRU = 3 };
+enum SmMode : int { SM_STORE = 0, SM_RESIDUAL = 1, SM_SWIGLU = 2, SM_MINGRU = 3, SM_SPLIT_GLU = 4 };
 
+// split_glu has two kinds of tiles: first those of the plain rows (one part of 64 channels), then those of the gated unit.
 template <int MODE> struct SmTile {
-  static constexpr int PARTS = MODE == SM_SWIGLU ? 2 : (MODE == SM_MINGRU ? 3 : 1);
-  static constexpr int CH = MODE == SM_SWIGLU ? 32 : (MODE == SM_MINGRU ? 16 : 64);  // channels per tile
+  static constexpr int PARTS = MODE == SM_SWIGLU || MODE == SM_SPLIT_GLU ? 2 : (MODE == SM_MINGRU ? 3 : 1);
+  static constexpr int CH = PARTS == 2 ? 32 : (MODE == SM_MINGRU ? 16 : 64);  // channels per tile
   static constexpr int COLS = PARTS * CH;
   static constexpr int NT = COLS / 8;
   static constexpr int STAGE = NT * 2 * 32;  // uint4: two pieces of NT weight rows per lane
@@ -51,8 +57,18 @@ struct SmParams {
   const int* tokens;
   const __nv_bfloat16* table;
   int vocab;
-  const float *alpha, *nw, *nb;
+  const float *alpha, *nw, *nb;  // DyT; alpha null: h = x * nw and the sums of squares
   __nv_bfloat16* h;
+  float* sumsq_out;  // (M, column tiles)
+  // store / split_glu: sums of squares of the rows of a half-done norm, (M, sumsq_parts), or null
+  const float* sumsq;
+  int sumsq_parts;
+  float eps;
+  // split_glu: y holds the plain results, z the unit's
+  int cols;
+  __nv_bfloat16* z;
+  long long ldz;
+  float limit, slope, shift;
   // min_gru
   const float *bz, *bu;
   float* state;
@@ -78,12 +94,21 @@ __device__ __forceinline__ float sigmoid_f(float v) { return 1.f / (1.f + expf(-
 __device__ __forceinline__ float silu_f(float v) { return v / (1.f + expf(-v)); }
 
 // Four channels c .. c + 3 of row r (those below `channels`). All loads come before the first store: their latencies overlap.
+// Returns the sum of squares of what it wrote to the residual stream.
 template <int MODE>
-__device__ __forceinline__ void sm_epilogue(const SmParams& p, int r, int c, const float (&v)[SmTile<MODE>::PARTS][4], int channels) {
+__device__ __forceinline__ float sm_epilogue(const SmParams& p, int r, int c, const float (&v)[SmTile<MODE>::PARTS][4], int channels,
+                                             bool unit) {
   constexpr int LAST = SmTile<MODE>::PARTS - 1;
   const int n = min(4, channels - c);
+  float sq = 0.f;
   const long long at = (long long)r * channels + c, yat = (long long)r * p.ldy + c;
-  if (MODE == SM_STORE) {
+  if (MODE == SM_SPLIT_GLU && unit) {
+#pragma unroll
+    for (int e = 0; e < 4; ++e)
+      if (e < n)
+        p.z[(long long)r * p.ldz + c + e] =
+            __float2bfloat16_rn(xl_clamped_glu_value(v[0][e], v[LAST][e], p.limit, p.slope, p.shift));
+  } else if (MODE == SM_STORE || MODE == SM_SPLIT_GLU) {
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       if (e < n) {
@@ -100,7 +125,7 @@ __device__ __forceinline__ void sm_epilogue(const SmParams& p, int r, int c, con
       const int k = e < n ? e : 0;
       x[e] = p.x[at + k];
       add[e] = row ? __bfloat162float(row[k]) : 0.f;
-      nw[e] = p.alpha ? p.nw[c + k] : 0.f;
+      nw[e] = p.nw ? p.nw[c + k] : 0.f;
       nb[e] = p.alpha ? p.nb[c + k] : 0.f;
     }
 #pragma unroll
@@ -108,7 +133,9 @@ __device__ __forceinline__ void sm_epilogue(const SmParams& p, int r, int c, con
       if (e < n) {
         const float s = x[e] + p.mult * v[0][e] + add[e];
         p.x[at + e] = s;
+        sq += s * s;
         if (p.alpha) p.h[at + e] = __float2bfloat16_rn(tanhf(alpha * s) * nw[e] + nb[e]);
+        else if (p.nw) p.h[at + e] = __float2bfloat16_rn(s * nw[e]);
       }
     }
   } else if (MODE == SM_SWIGLU) {
@@ -138,6 +165,7 @@ __device__ __forceinline__ void sm_epilogue(const SmParams& p, int r, int c, con
       }
     }
   }
+  return sq;
 }
 
 // Contiguous ranges of items: the first `rem` CTAs take per + 1 items, the others per.
@@ -157,11 +185,14 @@ __global__ void __launch_bounds__(SM_WARPS * 32, SM_CTAS_PER_SM) linear_small_m_
   extern __shared__ uint4 ring_all[];
   __shared__ float red[SM_WARPS][16][COLS + 1];
   __shared__ unsigned int finish;
+  __shared__ float row_scale[16];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int quad = lane >> 2, j = lane & 3;
-  const int channels = p.N / PARTS;
   const int chunks = (p.K + SM_KC - 1) / SM_KC;
-  const int n_tiles = (channels + CH - 1) / CH;
+  // tiles [0, plain) have one part of COLS channels (split_glu only), the others PARTS parts of CH
+  const int plain = MODE == SM_SPLIT_GLU ? (p.cols + COLS - 1) / COLS : 0;
+  const int channels = MODE == SM_SPLIT_GLU ? (p.N - p.cols) / PARTS : p.N / PARTS;
+  const int n_tiles = plain + (channels + CH - 1) / CH;
   const int total = n_tiles * chunks;
   const SmRanges ranges{total / (int)gridDim.x, total % (int)gridDim.x};
   int item = ranges.begin(blockIdx.x);
@@ -195,9 +226,18 @@ __global__ void __launch_bounds__(SM_WARPS * 32, SM_CTAS_PER_SM) linear_small_m_
       uint4* dst = ring + buf * L::STAGE + lane;
 #pragma unroll
       for (int t = 0; t < NT; ++t) {
-        const int col = t * 8 + quad, part = col / CH, n = c.tile * CH + col % CH;
-        const bool row_on = n < channels;
-        const __nv_bfloat16* src = p.w + ((long long)part * channels + (row_on ? n : 0)) * p.K;
+        const int col = t * 8 + quad;
+        bool row_on;
+        long long w_row;
+        if (MODE == SM_SPLIT_GLU && c.tile < plain) {
+          w_row = c.tile * COLS + col;
+          row_on = w_row < p.cols;
+        } else {
+          const int n = (c.tile - plain) * CH + col % CH;
+          row_on = n < channels;
+          w_row = (MODE == SM_SPLIT_GLU ? p.cols : 0) + (long long)(col / CH) * channels + n;
+        }
+        const __nv_bfloat16* src = p.w + (row_on ? w_row : 0) * p.K;
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
           const bool on = row_on && k0 + e * 32 < p.K;
@@ -228,6 +268,14 @@ __global__ void __launch_bounds__(SM_WARPS * 32, SM_CTAS_PER_SM) linear_small_m_
   xl_grid_launch_dependents();
   uint4 a_lo[2], a_hi[2];
   load_a(cur, a_lo, a_hi);
+  if ((MODE == SM_STORE || MODE == SM_SPLIT_GLU) && p.sumsq) {  // read after the barriers of the first tile
+    for (int r = warp; r < p.M; r += SM_WARPS) {
+      float sq = 0.f;
+      for (int i = lane; i < p.sumsq_parts; i += 32) sq += p.sumsq[(long long)r * p.sumsq_parts + i];
+      sq = xl_warp_sum(sq);
+      if (lane == 0) row_scale[r] = 1.f / sqrtf(sq / p.K + p.eps);
+    }
+  }
   int buf = 0;
   while (item < item_end) {
     const int tile = item / chunks;
@@ -295,32 +343,51 @@ __global__ void __launch_bounds__(SM_WARPS * 32, SM_CTAS_PER_SM) linear_small_m_
         cta1 = ranges.owner(tile * chunks + chunks - 1);
         slot0 = ranges.begin(cta0) < tile * chunks ? 1 : 0;
       }
-      for (int i = threadIdx.x; i < p.M * (CH / 4); i += blockDim.x) {
-        const int r = i / (CH / 4), cc = (i % (CH / 4)) * 4, c = tile * CH + cc;
-        if (c >= channels) continue;
-        float v[PARTS][4];
+      const bool unit = tile >= plain;  // one part of COLS channels, or PARTS parts of CH
+      const int ch = MODE == SM_SPLIT_GLU && !unit ? COLS : CH, parts = MODE == SM_SPLIT_GLU && !unit ? 1 : PARTS;
+      const int end = MODE == SM_SPLIT_GLU && !unit ? p.cols : channels, per_row = ch / 4;
+      for (int i = threadIdx.x; i < p.M * per_row; i += blockDim.x) {
+        const int r = i / per_row, cc = (i % per_row) * 4, c = (unit ? tile - plain : tile) * ch + cc;
+        float sq = 0.f;
+        if (c < end) {
+          float v[PARTS][4];
 #pragma unroll
-        for (int q = 0; q < PARTS; ++q) {
-          const int col = q * CH + cc;
-          if (whole) {
+          for (int q = 0; q < PARTS; ++q) {
+            const int col = q * CH + cc;
+            if (MODE == SM_SPLIT_GLU && q >= parts) {
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-              v[q][e] = 0.f;
+              for (int e = 0; e < 4; ++e) v[q][e] = 0.f;
+            } else if (whole) {
 #pragma unroll
-              for (int w = 0; w < SM_WARPS; ++w) v[q][e] += red[w][r][col + e];
-            }
-          } else {
-            const float* base = p.slots + r * COLS + col;
-            float4 t = __ldcg(reinterpret_cast<const float4*>(base + ((long long)cta0 * 2 + slot0) * (16 * COLS)));
+              for (int e = 0; e < 4; ++e) {
+                v[q][e] = 0.f;
+#pragma unroll
+                for (int w = 0; w < SM_WARPS; ++w) v[q][e] += red[w][r][col + e];
+              }
+            } else {
+              const float* base = p.slots + r * COLS + col;
+              float4 t = __ldcg(reinterpret_cast<const float4*>(base + ((long long)cta0 * 2 + slot0) * (16 * COLS)));
 #pragma unroll 8
-            for (int k = cta0 + 1; k <= cta1; ++k) {
-              const float4 o = __ldcg(reinterpret_cast<const float4*>(base + (long long)k * 2 * (16 * COLS)));
-              t.x += o.x; t.y += o.y; t.z += o.z; t.w += o.w;
+              for (int k = cta0 + 1; k <= cta1; ++k) {
+                const float4 o = __ldcg(reinterpret_cast<const float4*>(base + (long long)k * 2 * (16 * COLS)));
+                t.x += o.x; t.y += o.y; t.z += o.z; t.w += o.w;
+              }
+              v[q][0] = t.x; v[q][1] = t.y; v[q][2] = t.z; v[q][3] = t.w;
             }
-            v[q][0] = t.x; v[q][1] = t.y; v[q][2] = t.z; v[q][3] = t.w;
+            if ((MODE == SM_STORE || MODE == SM_SPLIT_GLU) && p.sumsq) {
+#pragma unroll
+              for (int e = 0; e < 4; ++e) v[q][e] *= row_scale[r];
+            }
           }
+          sq = sm_epilogue<MODE>(p, r, c, v, end, unit);
         }
-        sm_epilogue<MODE>(p, r, c, v, channels);
+        if (MODE == SM_RESIDUAL && p.sumsq_out) {
+          // the 16 lanes of a half-warp hold one row; either all or none of them are here
+          const unsigned int half = 0xffffu << (lane & 16);
+#pragma unroll
+          for (int o = 8; o > 0; o >>= 1) sq += __shfl_xor_sync(half, sq, o);
+          if ((lane & 15) == 0) p.sumsq_out[(long long)r * n_tiles + tile] = sq;
+        }
       }
       if (!whole && threadIdx.x == 0) p.counters[tile] = 0;
     }
@@ -330,8 +397,10 @@ __global__ void __launch_bounds__(SM_WARPS * 32, SM_CTAS_PER_SM) linear_small_m_
 
 template <int MODE> int sm_launch(const SmParams& p, int sms, int max_tiles, cudaStream_t s) {
   using L = SmTile<MODE>;
-  if (p.N % L::PARTS) return -1;
-  const int channels = p.N / L::PARTS, chunks = (p.K + SM_KC - 1) / SM_KC, n_tiles = (channels + L::CH - 1) / L::CH;
+  const int paired = MODE == SM_SPLIT_GLU ? p.N - p.cols : p.N;
+  if (paired % L::PARTS) return -1;
+  const int plain = MODE == SM_SPLIT_GLU ? (p.cols + L::COLS - 1) / L::COLS : 0;
+  const int channels = paired / L::PARTS, chunks = (p.K + SM_KC - 1) / SM_KC, n_tiles = plain + (channels + L::CH - 1) / L::CH;
   if (n_tiles > max_tiles) return -1;
   static bool configured = false;
   if (!configured) {
@@ -361,14 +430,45 @@ int sm_check(const void* a, long long lda, const void* w, int M, int N, int K, c
 XL_API int xl_linear_small_m_slots(int sms) { return SM_CTAS_PER_SM * sms * 2 * 16 * 64; }
 
 // All: a (M, K) bf16 with row stride lda (a multiple of 8), w (N, K) bf16 contiguous, M <= 16, K a multiple of 8; returns -1
-// for arguments the kernel does not take. y (M, N) with row stride ldy, bf16 or fp32.
-XL_API int xl_linear_small_m(const void* a, long long lda, const void* w, void* y, long long ldy, int y_f32, int M, int N, int K,
-                             float* slots, unsigned int* counters, int max_tiles, int sms, cudaStream_t s) {
-  if (sm_check(a, lda, w, M, N, K, slots, counters) || !y) return -1;
+// for arguments the kernel does not take. y (M, N) with row stride ldy, bf16 or fp32. sumsq (M, sumsq_parts), or null: the rows
+// of y are multiplied by 1 / sqrt(sum of the row's sumsq / K + eps).
+XL_API int xl_linear_small_m(const void* a, long long lda, const void* w, void* y, long long ldy, int y_f32, const float* sumsq,
+                             int sumsq_parts, float eps, int M, int N, int K, float* slots, unsigned int* counters, int max_tiles,
+                             int sms, cudaStream_t s) {
+  if (sm_check(a, lda, w, M, N, K, slots, counters) || !y || (sumsq && sumsq_parts < 1)) return -1;
   SmParams p = {};
   p.a = (const __nv_bfloat16*)a; p.lda = lda; p.w = (const __nv_bfloat16*)w; p.M = M; p.N = N; p.K = K;
-  p.y = y; p.ldy = ldy; p.y_f32 = y_f32; p.slots = slots; p.counters = counters;
+  p.y = y; p.ldy = ldy; p.y_f32 = y_f32; p.sumsq = sumsq; p.sumsq_parts = sumsq_parts; p.eps = eps;
+  p.slots = slots; p.counters = counters;
   return sm_launch<SM_STORE>(p, sms, max_tiles, s);
+}
+
+// w rows [cols plain | F gate | F up], N = cols + 2F: y (M, cols) with row stride ldy and z (M, F) with row stride ldz, bf16;
+// sumsq as in xl_linear_small_m.
+XL_API int xl_linear_small_m_split_glu(const void* a, long long lda, const void* w, void* y, long long ldy, int cols, void* z,
+                                       long long ldz, float limit, float slope, float shift, const float* sumsq, int sumsq_parts,
+                                       float eps, int M, int N, int K, float* slots, unsigned int* counters, int max_tiles,
+                                       int sms, cudaStream_t s) {
+  if (sm_check(a, lda, w, M, N, K, slots, counters) || cols < 0 || cols > N || (cols && !y) || (cols < N && !z) ||
+      (sumsq && sumsq_parts < 1))
+    return -1;
+  SmParams p = {};
+  p.a = (const __nv_bfloat16*)a; p.lda = lda; p.w = (const __nv_bfloat16*)w; p.M = M; p.N = N; p.K = K;
+  p.y = y; p.ldy = ldy; p.cols = cols; p.z = (__nv_bfloat16*)z; p.ldz = ldz; p.limit = limit; p.slope = slope; p.shift = shift;
+  p.sumsq = sumsq; p.sumsq_parts = sumsq_parts; p.eps = eps; p.slots = slots; p.counters = counters;
+  return sm_launch<SM_SPLIT_GLU>(p, sms, max_tiles, s);
+}
+
+// x (M, N) fp32 += mult * a w^T; with nw, h (M, N) bf16 = x * nw and sumsq (M, ceil(N / 64)) = sums of x^2 over 64 columns.
+XL_API int xl_linear_small_m_residual_rms(const void* a, long long lda, const void* w, float* x, float mult, const float* nw,
+                                          void* h, float* sumsq, int M, int N, int K, float* slots, unsigned int* counters,
+                                          int max_tiles, int sms, cudaStream_t s) {
+  if (sm_check(a, lda, w, M, N, K, slots, counters) || !x || (nw && (!h || !sumsq))) return -1;
+  SmParams p = {};
+  p.a = (const __nv_bfloat16*)a; p.lda = lda; p.w = (const __nv_bfloat16*)w; p.M = M; p.N = N; p.K = K;
+  p.x = x; p.mult = mult; p.nw = nw; p.h = (__nv_bfloat16*)h; p.sumsq_out = nw ? sumsq : nullptr;
+  p.slots = slots; p.counters = counters;
+  return sm_launch<SM_RESIDUAL>(p, sms, max_tiles, s);
 }
 
 // x (M, N) fp32 += mult * a w^T (+ table[tokens]); with alpha, h (M, N) bf16 = tanh(alpha x) nw + nb.

@@ -2,7 +2,10 @@
 //   xl_embed_dyt        x = table[token] (fp32) and h = DyT(x), the first normalised activations
 //   xl_residual_dyt     x += mult * y (+ table[token]) and h = DyT(x) of the updated stream, one pass
 //   xl_select_dyt       DyT of selected rows of the stream (the rows whose logits are asked for)
+//   xl_stream_rms       x = scale * table[token], or x += mult * y, and h = the RMS norm of the updated stream, one pass
+//   xl_select_rms       RMS norm of selected rows of the stream
 //   xl_swiglu_packed    silu(gate) * up on rows [gate | up]
+//   xl_clamped_glu      g * sigmoid(slope g) * (u + shift) of clamped gate and up columns of wider rows
 //   xl_min_gru          gated linear recurrence S_t = (1 - z_t) S_{t-1} + z_t c_t over a portion of every sequence
 //   xl_advance_by       pos[b] += count[b]
 // Dynamic Tanh (DyT): tanh(alpha * x) * w + b, element by element, so it folds into whatever produced x.
@@ -96,6 +99,106 @@ __global__ void __launch_bounds__(256)
   src = src < 0 ? 0 : (src >= x_rows ? x_rows - 1 : src);
   for (int c = threadIdx.x; c < cols; c += blockDim.x)
     h[r * cols + c] = xl_from_float<T>(tanhf(alpha * x[src * cols + c]) * n.w[c] + n.b[c]);
+}
+
+// ---- RMS norm: one CTA per row, the row in registers between the sum of squares and the output --------------------------
+constexpr int RMS_THREADS = 256;
+
+// x (rows, cols) fp32 += mult * y, or without y: x = mult * table[token]; with w, h = x / sqrt(mean(x^2) + eps) * w.
+// NP packs of V columns per thread stay in registers; the columns of longer rows are read again.
+template <typename T, int V, int NP>
+__global__ void __launch_bounds__(RMS_THREADS)
+    stream_rms_kernel(float* __restrict__ x, const T* __restrict__ y, float mult, const int* __restrict__ tokens,
+                      const T* __restrict__ table, int vocab, const float* __restrict__ w, float eps, T* __restrict__ h, int cols) {
+  __shared__ float red[32];
+  const long long row = blockIdx.x;
+  float* xr = x + row * cols;
+  const T* src = y ? y + row * cols : table + (long long)min(max(tokens[row], 0), vocab - 1) * cols;
+  const int step = blockDim.x * V, c0 = threadIdx.x * V;
+  float keep[NP][V], sq = 0.f;
+#pragma unroll
+  for (int i = 0; i < NP; ++i) {
+    const int c = c0 + i * step;
+    if (c < cols) {
+      float d[V];
+      load_pack<T, V>(src + c, d);
+      if (y) load_pack<float, V>(xr + c, keep[i]);
+#pragma unroll
+      for (int e = 0; e < V; ++e) {
+        keep[i][e] = y ? keep[i][e] + mult * d[e] : mult * d[e];
+        sq += keep[i][e] * keep[i][e];
+      }
+      store_pack<float, V>(xr + c, keep[i]);
+    }
+  }
+  for (int c = c0 + NP * step; c < cols; c += step) {
+    float d[V], v[V];
+    load_pack<T, V>(src + c, d);
+    if (y) load_pack<float, V>(xr + c, v);
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+      v[e] = y ? v[e] + mult * d[e] : mult * d[e];
+      sq += v[e] * v[e];
+    }
+    store_pack<float, V>(xr + c, v);
+  }
+  if (!w) return;
+  const float f = 1.f / sqrtf(xl_block_sum(sq, red) / cols + eps);
+  T* hr = h + row * cols;
+#pragma unroll
+  for (int i = 0; i < NP; ++i) {
+    const int c = c0 + i * step;
+    if (c < cols) {
+      float g[V];
+      load_pack<float, V>(w + c, g);
+#pragma unroll
+      for (int e = 0; e < V; ++e) g[e] *= keep[i][e] * f;
+      store_pack<T, V>(hr + c, g);
+    }
+  }
+  for (int c = c0 + NP * step; c < cols; c += step) {
+    float g[V], v[V];
+    load_pack<float, V>(w + c, g);
+    load_pack<float, V>(xr + c, v);  // written by this thread
+#pragma unroll
+    for (int e = 0; e < V; ++e) g[e] *= v[e] * f;
+    store_pack<T, V>(hr + c, g);
+  }
+}
+
+// h[r] = RMS norm of x[r * stride + idx[r] - offset]
+template <typename T>
+__global__ void __launch_bounds__(RMS_THREADS)
+    select_rms_kernel(const float* __restrict__ x, const int* __restrict__ idx, int stride, int offset, long long x_rows,
+                      const float* __restrict__ w, float eps, T* __restrict__ h, int cols) {
+  __shared__ float red[32];
+  const long long r = blockIdx.x;
+  long long src = r * stride + idx[r] - offset;
+  src = src < 0 ? 0 : (src >= x_rows ? x_rows - 1 : src);
+  const float* xr = x + src * cols;
+  float sq = 0.f;
+  for (int c = threadIdx.x; c < cols; c += blockDim.x) sq += xr[c] * xr[c];
+  const float f = 1.f / sqrtf(xl_block_sum(sq, red) / cols + eps);
+  for (int c = threadIdx.x; c < cols; c += blockDim.x) h[r * cols + c] = xl_from_float<T>(xr[c] * f * w[c]);
+}
+
+// gate: columns [0, F) of rows of stride ldg, up: the F columns after them; y: F columns of rows of stride ldy.
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+    clamped_glu_kernel(const T* __restrict__ gate, long long ldg, T* __restrict__ y, long long ldy, long long rows, int F,
+                       float limit, float slope, float shift) {
+  const int per_row = F / V;
+  const long long total = rows * per_row;
+  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
+    const long long row = i / per_row;
+    const int c = (int)(i - row * per_row) * V;
+    float g[V], u[V];
+    load_pack<T, V>(gate + row * ldg + c, g);
+    load_pack<T, V>(gate + row * ldg + F + c, u);
+#pragma unroll
+    for (int e = 0; e < V; ++e) g[e] = xl_clamped_glu_value(g[e], u[e], limit, slope, shift);
+    store_pack<T, V>(y + row * ldy + c, g);
+  }
 }
 
 template <typename T, int V>
@@ -260,7 +363,59 @@ int launch_stream(float* x, const void* y, float mult, const int* tokens, const 
   return (int)cudaGetLastError();
 }
 
+template <typename T, int V>
+int launch_rms(float* x, const void* y, float mult, const int* tokens, const void* table, int vocab, const float* w, float eps,
+               void* h, long long rows, int cols, cudaStream_t s) {
+  const int packs = (cols + V - 1) / V;
+  const int threads = packs >= RMS_THREADS ? RMS_THREADS : (packs + 31) / 32 * 32;
+#define XL_RMS(NP)                                                                                                         \
+  stream_rms_kernel<T, V, NP><<<(unsigned)rows, threads, 0, s>>>(x, (const T*)y, mult, tokens, (const T*)table, vocab, w,    \
+                                                                 eps, (T*)h, cols)
+  if (packs <= RMS_THREADS) XL_RMS(1);
+  else if (packs <= 4 * RMS_THREADS) XL_RMS(4);
+  else XL_RMS(8);
+#undef XL_RMS
+  return (int)cudaGetLastError();
+}
+
 }  // namespace
+
+// x (rows, cols) fp32; y, h, table of type `dtype`. y null: x = mult * table[tokens] (embedding), else x += mult * y. w null: no
+// norm (h unused), else h = x / sqrt(mean(x^2) + eps) * w, w fp32. All base pointers 16-byte aligned.
+XL_API int xl_stream_rms(float* x, const void* y, float mult, const int* tokens, const void* table, int vocab, const float* w,
+                         float eps, void* h, long long rows, int cols, int dtype, cudaStream_t s) {
+  if (rows < 1 || rows > 0x7fffffffLL || cols < 1 || (!y && (!table || !tokens || vocab < 1)) || (w && !h)) return -1;
+  XL_DISPATCH_DTYPE(dtype, T, {
+    return cols % 4 == 0 ? launch_rms<T, 4>(x, y, mult, tokens, table, vocab, w, eps, h, rows, cols, s)
+                         : launch_rms<T, 1>(x, y, mult, tokens, table, vocab, w, eps, h, rows, cols, s);
+  });
+  return (int)cudaGetLastError();
+}
+
+XL_API int xl_select_rms(const float* x, const int* idx, int stride, int offset, long long x_rows, const float* w, float eps,
+                         void* h, int rows, int cols, int dtype, cudaStream_t s) {
+  if (rows < 1 || cols < 1 || x_rows < 1 || !w) return -1;
+  XL_DISPATCH_DTYPE(dtype, T, {
+    select_rms_kernel<T><<<rows, RMS_THREADS, 0, s>>>(x, idx, stride, offset, x_rows, w, eps, (T*)h, cols);
+  });
+  return (int)cudaGetLastError();
+}
+
+// gate: first of 2F columns [gate | up] inside rows of stride ldg; y: first of F columns inside rows of stride ldy.
+XL_API int xl_clamped_glu(const void* gate, long long ldg, void* y, long long ldy, long long rows, int F, float limit,
+                          float slope, float shift, int dtype, cudaStream_t s) {
+  if (rows < 1 || F < 1 || ldg < 2LL * F || ldy < F) return -1;
+  XL_DISPATCH_DTYPE(dtype, T, {
+    constexpr int V = 16 / sizeof(T);
+    if (F % V == 0 && ldg % V == 0 && ldy % V == 0 && (((uintptr_t)gate | (uintptr_t)y) & 15) == 0)
+      clamped_glu_kernel<T, V><<<xl_grid_for(rows * (F / V), 256), 256, 0, s>>>((const T*)gate, ldg, (T*)y, ldy, rows, F, limit,
+                                                                               slope, shift);
+    else
+      clamped_glu_kernel<T, 1><<<xl_grid_for(rows * F, 256), 256, 0, s>>>((const T*)gate, ldg, (T*)y, ldy, rows, F, limit,
+                                                                         slope, shift);
+  });
+  return (int)cudaGetLastError();
+}
 
 // x (rows, cols) fp32; y, h, table of type `dtype`. y null: x = table[tokens] (embedding). table null: no row is added.
 // alpha null: no norm (h unused), else h = tanh(alpha x) w + b. All base pointers 16-byte aligned.

@@ -162,6 +162,24 @@ __device__ __forceinline__ uint4 pack8_16bit(const float* v, bool is_fp16) {
   return make_uint4(w[0], w[1], w[2], w[3]);
 }
 
+// Attention weights (N per thread, one query row each) as the A operand of a later product in TMEM, two bf16 numbers per weight:
+// the rounded values in columns [0, N / 2), their rounding errors in [N / 2, N).
+template <int N> __device__ __forceinline__ void store_split_weights(uint32_t tmem, const float (&s)[N]) {
+#pragma unroll
+  for (int ch = 0; ch < N / 32; ++ch) {
+    uint32_t hi[16], err[16];
+#pragma unroll
+    for (int i = 0; i < 16; ++i) {
+      const float x = s[ch * 32 + 2 * i], y = s[ch * 32 + 2 * i + 1];
+      asm("cvt.rn.bf16x2.f32 %0, %1, %2;" : "=r"(hi[i]) : "f"(y), "f"(x));
+      const float ex = x - __uint_as_float(hi[i] << 16), ey = y - __uint_as_float(hi[i] & 0xffff0000u);
+      asm("cvt.rn.bf16x2.f32 %0, %1, %2;" : "=r"(err[i]) : "f"(ey), "f"(ex));
+    }
+    tmem_st_32x32b_x16(tmem + ch * 16, hi);
+    tmem_st_32x32b_x16(tmem + N / 2 + ch * 16, err);
+  }
+}
+
 // one 32-byte store to global memory (the address must be 32-byte aligned)
 __device__ __forceinline__ void st_global_v8(void* ptr, const uint4& a, const uint4& b) {
   asm volatile("st.global.v8.b32 [%0], {%1, %2, %3, %4, %5, %6, %7, %8};" ::"l"(ptr), "r"(a.x), "r"(a.y), "r"(a.z), "r"(a.w),
@@ -201,6 +219,20 @@ static inline EncodeTiledFn get_encode_fn() {
     return nullptr;
   fn = (EncodeTiledFn)ptr;
   return fn;
+}
+
+// 2-D map over a row-major bf16 matrix, boxes of {64, box_rows}, 128-byte swizzle
+static inline int make_map_bf16(CUtensorMap* map, const void* ptr, long long rows, long long cols, long long ld, int box_rows) {
+  EncodeTiledFn fn = get_encode_fn();
+  if (!fn) return -2;
+  cuuint64_t dims[2] = {(cuuint64_t)cols, (cuuint64_t)rows};
+  cuuint64_t strides[1] = {(cuuint64_t)ld * 2};
+  cuuint32_t box[2] = {64, (cuuint32_t)box_rows};
+  cuuint32_t estr[2] = {1, 1};
+  const CUresult r = fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (void*)ptr, dims, strides, box, estr,
+                        CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                        CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  return r == CUDA_SUCCESS ? 0 : -3;
 }
 
 }  // namespace xl_tc

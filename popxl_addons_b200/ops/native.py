@@ -218,7 +218,13 @@ def check_gemm_errors():
                      43: "differential attention: key / value stage was never released",
                      44: "differential attention: scores never completed",
                      45: "differential attention: probabilities never arrived",
-                     46: "differential attention: output accumulation never completed"}
+                     46: "differential attention: output accumulation never completed",
+                     51: "window attention: query tiles never arrived",
+                     52: "window attention: key / value tile never arrived",
+                     53: "window attention: key / value stage was never released",
+                     54: "window attention: scores never completed",
+                     55: "window attention: probabilities never arrived",
+                     56: "window attention: output accumulation never completed"}
             raise RuntimeError(f"tcgen05 GEMM on cuda:{idx} gave up waiting: {names.get(code, code)}")
 
 

@@ -3,6 +3,7 @@
 import torch
 
 from ..xl.opdef import native
+from ..xl.ops.sequence import SUMSQ_BLOCK
 from .native import (_CODE, _c_f, _c_int, _c_ll, _c_p, _check, _count, _ok, _sig, _sms, _stream, gemm,
                      gemm_error_flag)
 
@@ -20,9 +21,24 @@ _diff_decode = _sig("xl_diff_attn_decode", _c_p, _c_ll, _c_p, _c_p, _c_p, _c_p, 
                     _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_f, _c_f, _c_f, _c_int, _c_p, _c_p, _c_p)
 _diff_tcgen05 = _sig("xl_diff_attn_tcgen05", _c_p, _c_ll, _c_p, _c_p, _c_p, _c_ll, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int,
                      _c_int, _c_int, _c_int, _c_int, _c_f, _c_f, _c_f, _c_p, _c_p)
+_stream_rms = _sig("xl_stream_rms", _c_p, _c_p, _c_f, _c_p, _c_p, _c_int, _c_p, _c_f, _c_p, _c_ll, _c_int, _c_int, _c_p)
+_select_rms = _sig("xl_select_rms", _c_p, _c_p, _c_int, _c_int, _c_ll, _c_p, _c_f, _c_p, _c_int, _c_int, _c_int, _c_p)
+_clamped_glu = _sig("xl_clamped_glu", _c_p, _c_ll, _c_p, _c_ll, _c_ll, _c_int, _c_f, _c_f, _c_f, _c_int, _c_p)
+_qk_norm_append = _sig("xl_qk_norm_append", _c_p, _c_ll, _c_p, _c_p, _c_p, _c_p, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int,
+                       _c_int, _c_int, _c_int, _c_f, _c_int, _c_p)
+_WINDOW_ARGS = (_c_p, _c_p, _c_p, _c_p, _c_ll, _c_p, _c_ll, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
+                _c_int, _c_int, _c_f, _c_f)
+_window_general = _sig("xl_window_attn_general", *_WINDOW_ARGS, _c_int, _c_p)
+_window_tcgen05 = _sig("xl_window_attn_tcgen05", *_WINDOW_ARGS, _c_p, _c_p)
+_window_decode = _sig("xl_window_attn_decode", _c_p, _c_ll, _c_p, _c_p, _c_p, _c_p, _c_p, _c_ll, _c_p, _c_p, _c_int, _c_int, _c_int,
+                      _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_f, _c_f, _c_f, _c_int, _c_p, _c_p, _c_p)
 _small_m_slots = _sig("xl_linear_small_m_slots", _c_int)
 _SMALL_TAIL = (_c_int, _c_int, _c_int, _c_p, _c_p, _c_int, _c_int, _c_p)
-_small_store = _sig("xl_linear_small_m", _c_p, _c_ll, _c_p, _c_p, _c_ll, _c_int, *_SMALL_TAIL)
+_SUMSQ = (_c_p, _c_int, _c_f)  # sums of squares of a deferred norm, parts per row, eps
+_small_store = _sig("xl_linear_small_m", _c_p, _c_ll, _c_p, _c_p, _c_ll, _c_int, *_SUMSQ, *_SMALL_TAIL)
+_small_split_glu = _sig("xl_linear_small_m_split_glu", _c_p, _c_ll, _c_p, _c_p, _c_ll, _c_int, _c_p, _c_ll, _c_f, _c_f, _c_f, *_SUMSQ,
+                        *_SMALL_TAIL)
+_small_residual_rms = _sig("xl_linear_small_m_residual_rms", _c_p, _c_ll, _c_p, _c_p, _c_f, _c_p, _c_p, _c_p, *_SMALL_TAIL)
 _small_residual = _sig("xl_linear_small_m_residual", _c_p, _c_ll, _c_p, _c_p, _c_f, _c_p, _c_p, _c_int, _c_p, _c_p, _c_p, _c_p,
                        *_SMALL_TAIL)
 _small_swiglu = _sig("xl_linear_small_m_swiglu", _c_p, _c_ll, _c_p, _c_p, *_SMALL_TAIL)
@@ -74,22 +90,31 @@ def _i32(*ts) -> bool:
     return all(t is None or (t.is_cuda and t.is_contiguous() and t.dtype == torch.int32) for t in ts)
 
 
-def product(a, weight, out_dtype=None):
+def _sumsq_args(sumsq, eps):
+    return (_ptr(sumsq), sumsq.shape[1] if sumsq is not None else 0, float(eps))
+
+
+def product(a, weight, out_dtype=None, sumsq=None, eps=0.0):
     """`a (n, K) @ weight (N, K)^T` with 32-bit accumulation: the tcgen05 GEMM for 16-bit operands, the vendor product for
-    sizes it does not take and for 32-bit models."""
+    sizes it does not take and for 32-bit models. `sumsq`: `a` is half of a deferred norm (few rows only, else
+    NotImplemented)."""
     out_dtype = out_dtype or a.dtype
     if a.dtype != torch.float32:
         if _small(a, weight) and out_dtype in (torch.bfloat16, torch.float32):
             y = torch.empty((a.shape[0], weight.shape[0]), dtype=out_dtype, device=a.device)
             if _small_ok(_small_store(a.data_ptr(), a.stride(0), weight.data_ptr(), y.data_ptr(), y.stride(0),
-                                      int(out_dtype == torch.float32), *_small_tail(a, weight.shape[0], weight)),
-                         "linear_small_m"):
+                                      int(out_dtype == torch.float32), *_sumsq_args(sumsq, eps),
+                                      *_small_tail(a, weight.shape[0], weight)), "linear_small_m"):
                 return y
+        if sumsq is not None:
+            return NotImplemented
         y = gemm(a, weight.t(), out_dtype=out_dtype)
         if y is not NotImplemented:
             return y
         y = torch.mm(a, weight.t())
         return y if y.dtype == out_dtype else y.to(out_dtype)
+    if sumsq is not None:
+        return NotImplemented
     if torch.backends.cuda.matmul.allow_tf32:
         raise RuntimeError("32-bit models need true fp32 matrix products: set torch.backends.cuda.matmul.allow_tf32 = False")
     return torch.mm(a, weight.t()).to(out_dtype)
@@ -152,8 +177,8 @@ def select_dyt_cuda(x, idx, alpha, w, b, stride, offset, out_dtype):
 
 
 @native("linear_rows")
-def linear_rows_cuda(a, weight, out_dtype):
-    return product(a, weight, out_dtype)
+def linear_rows_cuda(a, weight, *sumsq, out_dtype, eps=0.0):
+    return product(a, weight, out_dtype, sumsq[0] if sumsq else None, eps)
 
 
 @native("linear_swiglu")
@@ -237,6 +262,125 @@ def diff_attention_cuda(qkv, cos, sin, kc, vc, pos, count, lam, T, heads, rotary
     _check(rc, "diff_attn_general")
     _count("diff_attn_general")
     return out
+
+
+def stream_rms(x, y, mult, tokens, table, w, eps, out_dtype):
+    """One pass over the residual stream: `x += mult * y`, or `x = mult * table[tokens]` without `y`; returns the RMS norm of
+    it when its factors `w` are given."""
+    rows, cols = y.shape[0] if y is not None else tokens.numel(), x.shape[1]
+    if not _ok(x, y, table, w) or not _f32(x, w) or not _i32(tokens) or rows > x.shape[0]:
+        return NotImplemented
+    h = torch.empty((rows, cols), dtype=out_dtype, device=x.device) if w is not None else None
+    rc = _stream_rms(x.data_ptr(), _ptr(y), float(mult), _ptr(tokens), _ptr(table), table.shape[0] if table is not None else 0,
+                     _ptr(w), float(eps), _ptr(h), rows, cols, _CODE[out_dtype], _stream())
+    if rc == -1:
+        return NotImplemented
+    _check(rc, "stream_rms")
+    _count("stream_rms")
+    return h if w is not None else ()
+
+
+@native("embed_rms_")
+def embed_rms_cuda(x, tokens, table, w, scale, eps):
+    return stream_rms(x, None, scale, tokens.reshape(-1), table, w, eps, table.dtype)
+
+
+@native("linear_residual_rms_")
+def linear_residual_rms_cuda(x, a, weight, *norm, mult, eps, deferred):
+    w = norm[0] if norm else None
+    if (_small(a, weight) and (deferred or w is None) and _f32(x, w) and x.is_contiguous() and a.shape[0] <= x.shape[0]):
+        n, cols = a.shape[0], x.shape[1]
+        h = torch.empty((n, cols), dtype=a.dtype, device=a.device) if deferred else None
+        sumsq = torch.empty((n, -(-cols // SUMSQ_BLOCK)), dtype=torch.float32, device=a.device) if deferred else None
+        rc = _small_residual_rms(a.data_ptr(), a.stride(0), weight.data_ptr(), x.data_ptr(), float(mult), _ptr(w), _ptr(h),
+                                 _ptr(sumsq), *_small_tail(a, weight.shape[0], weight))
+        if _small_ok(rc, "linear_small_m_residual"):
+            return (h, sumsq) if deferred else ()
+    if deferred:
+        return NotImplemented
+    return stream_rms(x, product(a, weight), mult, None, None, w, eps, a.dtype)
+
+
+@native("select_rms")
+def select_rms_cuda(x, idx, w, stride, offset, eps, out_dtype):
+    if not _ok(x) or not _f32(x, w) or not _i32(idx):
+        return NotImplemented
+    h = torch.empty((idx.shape[0], x.shape[1]), dtype=out_dtype, device=x.device)
+    rc = _select_rms(x.data_ptr(), idx.data_ptr(), stride, offset, x.shape[0], w.data_ptr(), float(eps), h.data_ptr(),
+                     idx.shape[0], x.shape[1], _CODE[out_dtype], _stream())
+    if rc == -1:
+        return NotImplemented
+    _check(rc, "select_rms")
+    _count("select_rms")
+    return h
+
+
+@native("linear_split_glu")
+def linear_split_glu_cuda(h, weight, *sumsq, cols, lead, limit, slope, shift, eps=0.0):
+    n, N = h.shape[0], weight.shape[0]
+    f, sq = (N - cols) // 2, sumsq[0] if sumsq else None
+    joint = torch.empty((n, lead + f), dtype=h.dtype, device=h.device)
+    unit = joint.data_ptr() + lead * joint.element_size()
+    if _small(h, weight):
+        proj = torch.empty((n, cols), dtype=h.dtype, device=h.device)
+        rc = _small_split_glu(h.data_ptr(), h.stride(0), weight.data_ptr(), proj.data_ptr(), cols, cols, unit, lead + f, limit,
+                              slope, shift, *_sumsq_args(sq, eps), *_small_tail(h, N, weight))
+        if _small_ok(rc, "linear_small_m_split_glu"):
+            return proj, joint
+    y = product(h, weight, None, sq, eps)
+    if y is NotImplemented:
+        return NotImplemented
+    if f:
+        rc = _clamped_glu(y.data_ptr() + cols * y.element_size(), N, unit, lead + f, n, f, limit, slope, shift, _CODE[h.dtype],
+                          _stream())
+        _check(rc, "clamped_glu")
+        _count("clamped_glu")
+    return y[:, :cols], joint
+
+
+@native("window_attention_")
+def window_attention_cuda(proj, q_norm, k_norm, kc, vc, pos, count, joint, T, heads, window, keep_first, scale, sink, eps):
+    B, G, smax, dim = kc.shape
+    vdim = vc.shape[-1]
+    plain = (heads + G) * dim + G * vdim
+    gated = proj.shape[1] > plain
+    if not _ok(kc, vc, joint) or not (proj.dtype == kc.dtype == vc.dtype == joint.dtype) or not _f32(q_norm, k_norm):
+        return NotImplemented
+    if not _i32(pos, count) or proj.stride(1) != 1 or proj.shape != (B * T, plain + (heads * vdim if gated else 0)):
+        return NotImplemented
+    code, s, ld, ldo = _CODE[proj.dtype], _stream(), proj.stride(0), joint.stride(0)
+    sink = float("-inf") if sink is None else sink
+    if T == 1 and proj.dtype == torch.bfloat16:
+        units = B * G * ((heads // G + 15) // 16)
+        longest = min(smax, window + keep_first) if window else smax
+        splits = max(1, min(2 * _sms(proj.device) // units, (longest + 63) // 64, 64))  # one wave, two CTAs per SM
+        counters = _scratch(proj.device)[2]
+        part = torch.empty(units * splits * 16 * (vdim + 2), dtype=torch.float32, device=proj.device) if splits > 1 else None
+        if units <= counters.numel():
+            rc = _window_decode(proj.data_ptr(), ld, q_norm.data_ptr(), k_norm.data_ptr(), kc.data_ptr(), vc.data_ptr(),
+                                joint.data_ptr(), ldo, pos.data_ptr(), count.data_ptr(), B, heads, G, dim, vdim, smax, window,
+                                keep_first, int(gated), scale, sink, eps, splits, _ptr(part), counters.data_ptr(), s)
+            if _small_ok(rc, "window_attn_decode"):
+                return joint
+    qn = torch.empty((B, G, T, heads // G, dim), dtype=proj.dtype, device=proj.device)
+    rc = _qk_norm_append(proj.data_ptr(), ld, q_norm.data_ptr(), k_norm.data_ptr(), qn.data_ptr(), kc.data_ptr(), vc.data_ptr(),
+                         pos.data_ptr(), count.data_ptr(), B, T, heads, G, dim, vdim, smax, eps, code, s)
+    if rc == -1:
+        return NotImplemented
+    _check(rc, "qk_norm_append")
+    _count("qk_norm_append")
+    args = (qn.data_ptr(), kc.data_ptr(), vc.data_ptr(), proj.data_ptr() + plain * proj.element_size() if gated else None, ld,
+            joint.data_ptr(), ldo, pos.data_ptr(), count.data_ptr(), B, T, heads, G, dim, vdim, smax, window, keep_first, scale,
+            sink)
+    if proj.dtype == torch.bfloat16:
+        rc = _window_tcgen05(*args, gemm_error_flag(proj.device).data_ptr(), s)
+        if rc >= 0:
+            _check(rc, "window_attn_tcgen05")
+            _count("window_attn_tcgen05")
+            return joint
+    _check(_window_general(*args, code, s), "window_attn_general")
+    _count("window_attn_general")
+    return joint
 
 
 @native("advance_by_")

@@ -21,11 +21,9 @@ def head_norm(x, w, eps):
 
 def window_mask(n, size=None, keep_first=0):
     """`(n, n)` bool: may query i look at key j."""
-    m = torch.zeros(n, n, dtype=torch.bool)
-    for i in range(n):
-        for j in range(i + 1):
-            m[i, j] = size is None or i - j < size or j < keep_first
-    return m
+    i, j = torch.arange(n)[:, None], torch.arange(n)[None, :]
+    near = torch.ones(n, n, dtype=torch.bool) if size is None else i - j < size
+    return (j <= i) & (near | (j < keep_first))
 
 
 def sink_weights(s):

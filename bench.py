@@ -221,22 +221,46 @@ def run_decode(args, standalone: bool = True):
     return 0
 
 
-SERVING_METRIC = "serving tokens/s Dunelix layers (bf16, batch 16, prompt 512, 64 new tokens, greedy)"
+SERVING_METRIC = "serving tokens/s {} layers (bf16, batch 16, prompt 512, 64 new tokens, greedy)"
 
-# name: width, feed-forward, recurrent width, query heads, key / value heads (two maps of 64, values of 128 per head)
+# name: width, feed-forward, recurrent width, query heads, key / value heads (of 128 features, or two maps of 64 with values
+# of 128)
 SERVING_SIZES = {"w2048": (2048, 5632, 2048, 16, 4), "w4096": (4096, 11008, 4096, 32, 8), "w8192": (8192, 22016, 8192, 64, 8)}
 
 
+def _dunelix_serving(C, F, R, H, G, vocab, layers, chunk):
+    """Dunelix of four layers, one letter each: r recurrent (minGRU), a differential attention."""
+    from popxl_addons_b200.models.dunelix import Dunelix, DunelixConfig
+
+    gru = {"type": "mingru", "mixer": {"width": R}, "mlp": {"ff": F, "kind": "dense"}}
+    att = {"type": "attention", "mlp": {"ff": F, "kind": "dense"},
+           "mixer": {"heads": H, "kv_heads": G, "dim": 64, "vdim": 128, "diff": 0.5, "scale": 0.125, "mask": {"size": chunk},
+                     "rot": {"base": 500000.0, "dims": 64,
+                             "scaling": {"factor": 16.0, "low": 1.0, "high": 4.0, "original": 4096}}}}
+    return Dunelix(DunelixConfig.from_dict({"vocab": vocab, "width": C, "norm": {"eps": 1e-6}, "residual_mult": 0.5,
+                                            "layers": [{"r": gru, "a": att}[k] for k in layers]}))
+
+
+def _zirunex_serving(C, F, H, G, vocab, window):
+    from popxl_addons_b200.models.zirunex import Zirunex, ZirunexConfig
+
+    layer = {"type": "attention", "mlp": {"ff": F, "kind": "dense", "limit": 7.0},
+             "mixer": {"heads": H, "kv_heads": G, "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+                       "mask": {"size": window, "keep_first": 4}}}
+    return Zirunex(ZirunexConfig.from_dict({"vocab": vocab, "width": C, "norm": {"eps": 1e-6}, "embedding": {"scale": 8.0},
+                                            "layers": [layer] * 4}))
+
+
 def run_serving(args):
-    """Prefill and decoding of Dunelix at sizes that resemble a real model's layers (four layers: three minGRU, one
-    differential attention with chunks of 8192; random weights), beside the GPT-J-style `DecoderGenerator` (int4 weights)
-    with as many parameters per layer. One step = one `generate` call: 16 prompts of 512 tokens and 64 new tokens. `value`
-    is the total of prompt and new tokens of the middle size per second of device time."""
+    """Prefill and decoding of a sequence model at sizes that resemble a real model's layers (four layers, random weights),
+    beside the closest other model with as many parameters per layer. `dunelix`: three minGRU and one differential attention
+    with chunks of 8192, beside the GPT-J-style `DecoderGenerator` (int4 weights). `zirunex`: four layers of attention with
+    windows of 256, beside Dunelix with four attention layers and chunks of 256. One step = one `generate` call: 16 prompts of
+    512 tokens and 64 new tokens. `value` is the total of prompt and new tokens of the middle size per second of device time."""
     import numpy as np
     import torch
 
     from popxl_addons_b200.models.decoder import DecoderConfig
-    from popxl_addons_b200.models.dunelix import Dunelix, DunelixConfig
     from popxl_addons_b200.models.generator import DecoderGenerator
     from popxl_addons_b200.models.sequence_generator import SequenceGenerator
     from popxl_addons_b200.ops import native
@@ -272,49 +296,60 @@ def run_serving(args):
         launches_total += native.LAUNCHES["count"] - before
         return dict(prefill_ms=pre / K, ms_per_decode_step=dec / K / (N - 1), e2e_ms=wall / K, clocks=clocks.summary())
 
-    for name, (C, F, R, H, G) in SERVING_SIZES.items():
-        if args.model != "gptj_6b" and args.model != name:
-            continue
-        gru = {"type": "mingru", "mixer": {"width": R}, "mlp": {"ff": F, "kind": "dense"}}
-        att = {"type": "attention", "mlp": {"ff": F, "kind": "dense"},
-               "mixer": {"heads": H, "kv_heads": G, "dim": 64, "vdim": 128, "diff": 0.5, "scale": 0.125, "mask": {"size": 8192},
-                         "rot": {"base": 500000.0, "dims": 64,
-                                 "scaling": {"factor": 16.0, "low": 1.0, "high": 4.0, "original": 4096}}}}
-        cfg = DunelixConfig.from_dict({"vocab": vocab, "width": C, "norm": {"eps": 1e-6}, "residual_mult": 0.5,
-                                       "layers": [gru, gru, att, gru]})
-        model = Dunelix(cfg)
+    def serve(model):
         gen = SequenceGenerator(model, batch=B, max_seq=P + N, max_portion=P, max_new_tokens=N, device="cuda",
                                 cuda_graphs=not args.no_cuda_graphs)
         gen.load(model.random_weights(0, gen.session.device))
-        ours = measure(gen, True)
-        del gen
+        return measure(gen, True)
+
+    design, window = {"dunelix": "Dunelix", "zirunex": "Zirunex"}[args.mode], 256
+    for name, (C, F, R, H, G) in SERVING_SIZES.items():
+        if args.model != "gptj_6b" and args.model != name:
+            continue
+        if design == "Dunelix":
+            model = _dunelix_serving(C, F, R, H, G, vocab, "rrar", 8192)
+            # two maps, half of the square; one attention layer
+            att_flops, kv = 4 * (64 + 128) * P * P / 2 * H, B * (P + N / 2) * G * 256 * 2
+        else:
+            model = _zirunex_serving(C, F, H, G, vocab, window)
+            pairs, seen = window * P - window * (window - 1) / 2, min(window + 4, P)
+            att_flops, kv = 4 * 2 * (128 + 128) * pairs * H, 4 * B * seen * G * 256 * 2
+        body = model.cfg.param_count() - 2 * vocab * C
+        ours = serve(model)
         _free_device_memory()
-        body = cfg.param_count() - 2 * vocab * C
-        ffn = max(128, int((body / 4 - 4 * C * C) / (2 * C)) // 128 * 128)
-        jcfg = DecoderConfig(family="gptj", layers=4, hidden=C, heads=C // 128, head_dim=128, rotary_dim=64, ffn=ffn,
-                             vocab_size=vocab, seq_len=P + N)
-        gen = DecoderGenerator(jcfg, B, P, N, group_size=64, device="cuda", seed=0, cuda_graphs=not args.no_cuda_graphs)
-        like = measure(gen, False)
-        del gen
+        if design == "Dunelix":
+            like_name, ffn = "gptj_int4", max(128, int((body / 4 - 4 * C * C) / (2 * C)) // 128 * 128)
+            jcfg = DecoderConfig(family="gptj", layers=4, hidden=C, heads=C // 128, head_dim=128, rotary_dim=64, ffn=ffn,
+                                 vocab_size=vocab, seq_len=P + N)
+            gen = DecoderGenerator(jcfg, B, P, N, group_size=64, device="cuda", seed=0, cuda_graphs=not args.no_cuda_graphs)
+            like, like_body = measure(gen, False), body
+            like_bytes = (body + vocab * C) * (0.5 + 4 / 64) + B * (P + N / 2) * 2 * C * 2
+            like_att = 2 * P * P * C
+            del gen
+        else:
+            like_name = "dunelix"
+            ffn = F + (body // 4 - C * (2 * (H + G) * 64 + (G + H) * 128 + 3 * F)) // (3 * C) // 64 * 64
+            other = _dunelix_serving(C, ffn, R, H, G, vocab, "aaaa", window)
+            like, like_body = serve(other), other.cfg.param_count() - 2 * vocab * C
+            # decoding sees half a chunk on average, prompts half of every chunk's square
+            like_bytes = (like_body + vocab * C) * 2 + 4 * B * (window / 2) * G * 256 * 2
+            like_att = 4 * 4 * (64 + 128) * P * window / 2 * H
         _free_device_memory()
-        att_flops = 4 * (64 + 128) * P * P / 2 * H  # two maps, half of the square
-        kv = 16 * (P + N / 2) * G * 256 * 2
         for rec, bytes_step, flops in ((ours, (body + vocab * C) * 2 + kv, 2.0 * B * P * body + B * att_flops),
-                                       (like, (body + vocab * C) * (0.5 + 4 / 64) + 16 * (P + N / 2) * 2 * C * 2,
-                                        2.0 * B * P * body + B * 2 * P * P * C)):
+                                       (like, like_bytes, 2.0 * B * P * like_body + B * like_att)):
             rec.update(prefill_tokens_per_s=B * P / rec["prefill_ms"] * 1e3, decode_tokens_per_s=B / rec["ms_per_decode_step"] * 1e3,
                        e2e_tokens_per_s=B * (P + N) / rec["e2e_ms"] * 1e3,
                        prefill_frac=flops / rec["prefill_ms"] / 1e9 / peaks["bf16_tflops"],
                        decode_frac=bytes_step / rec["ms_per_decode_step"] / 1e6 / peaks["hbm_gbs"])
-        records.append({"size": name, "width": C, "ff": F, "heads": H, "kv_heads": G, "params_body": body, "dunelix": ours,
-                        "gptj_int4": {**like, "ffn": ffn}})
-    mid = records[len(records) // 2]["dunelix"]
+        records.append({"size": name, "width": C, "ff": F, "heads": H, "kv_heads": G, "params_body": body, args.mode: ours,
+                        like_name: {**like, "ffn": ffn}})
+    mid = records[len(records) // 2][args.mode]
     ms = mid["prefill_ms"] + mid["ms_per_decode_step"] * (N - 1)
     print(json.dumps({
-        "impl": "ours", "metric": SERVING_METRIC, "value": B * (P + N) / ms * 1e3, "unit": "tokens/s", "n_gpus": 1, "steps": K,
-        "warmup": W, "ms_per_step": ms, "higher_is_better": True, "scaling": "weak", "vs_baseline": None, "dtype": "bf16",
-        "data": "synthetic (uniform random prompt ids, random weights)",
-        "config": {"model": "Dunelix, 4 layers", "global_batch": B, "seq_len": P + N, "parallelism": "1 GPU",
+        "impl": "ours", "metric": SERVING_METRIC.format(design), "value": B * (P + N) / ms * 1e3, "unit": "tokens/s", "n_gpus": 1,
+        "steps": K, "warmup": W, "ms_per_step": ms, "higher_is_better": True, "scaling": "weak", "vs_baseline": None,
+        "dtype": "bf16", "data": "synthetic (uniform random prompt ids, random weights)",
+        "config": {"model": f"{design}, 4 layers", "global_batch": B, "seq_len": P + N, "parallelism": "1 GPU",
                    "l2": "weights and activations of a step exceed the 126 MB L2; no flush needed"},
         "clocks": mid["clocks"], "gpu_launches": launches_total,
         "e2e": {"value": mid["e2e_tokens_per_s"], "unit": "tokens/s", "h2d_bytes_per_step": B * P * 4 + 2 * B * 4,
@@ -433,12 +468,12 @@ def main():
     ap.add_argument("--micro-batch-size", type=int, default=1)
     ap.add_argument("--layers", type=int, default=0, help="override the layer count (diagnostics only; such a run is "
                                                          "labelled and is not the headline configuration)")
-    ap.add_argument("--mode", default="train", choices=["train", "decode", "pipeline", "dunelix"],
+    ap.add_argument("--mode", default="train", choices=["train", "decode", "pipeline", "dunelix", "zirunex"],
                     help="train: the training step (default, headline), followed by the PyTorch arm of the same step and "
                          "the int4 decode benchmark as secondary records; decode: int4 greedy generation, TP over all "
                          "GPUs; pipeline: pipeline x data parallel training (--stages device slots per replica); "
-                         "dunelix: prefill and decoding of Dunelix layers at several sizes beside the int4 GPT-J "
-                         "generator (one GPU; --model w2048|w4096|w8192 runs one size)")
+                         "dunelix, zirunex: prefill and decoding of that design's layers at several sizes, beside the int4 "
+                         "GPT-J generator / beside Dunelix (one GPU; --model w2048|w4096|w8192 runs one size)")
     ap.add_argument("--tp", type=int, default=0, help="train mode: tensor-parallel width (default min(gpus, 4))")
     ap.add_argument("--stages", type=int, default=4, help="pipeline mode: device slots (GPUs) per replica")
     ap.add_argument("--sequence-parallel", action="store_true",
@@ -472,7 +507,7 @@ def main():
         return run_reference(args)
     if args.mode == "decode":
         return run_decode(args)
-    if args.mode == "dunelix":
+    if args.mode in ("dunelix", "zirunex"):
         return run_serving(args)
 
     import torch

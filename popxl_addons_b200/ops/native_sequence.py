@@ -353,7 +353,8 @@ def window_attention_cuda(proj, q_norm, k_norm, kc, vc, pos, count, joint, T, he
     if T == 1 and proj.dtype == torch.bfloat16:
         units = B * G * ((heads // G + 15) // 16)
         longest = min(smax, window + keep_first) if window else smax
-        splits = max(1, min(2 * _sms(proj.device) // units, (longest + 63) // 64, 64))  # one wave, two CTAs per SM
+        # one wave, two CTAs per SM; a slice of fewer keys costs more in the merge than it saves
+        splits = max(1, min(2 * _sms(proj.device) // units, (longest + 383) // 384, 64))
         counters = _scratch(proj.device)[2]
         part = torch.empty(units * splits * 16 * (vdim + 2), dtype=torch.float32, device=proj.device) if splits > 1 else None
         if units <= counters.numel():

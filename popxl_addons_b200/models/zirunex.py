@@ -2,10 +2,10 @@
 
     x = scale * embed[token];   every layer: h = norm(x), x += attention(h) + feed_forward(h);   logits = head(norm(x))
 
-Norms are RMS norms with weights around one. The attention has grouped heads with normalised queries and keys, no positions, a
-window next to the first tokens, which stay visible, a sink in the softmax, and a gate on its output; the feed-forward is a gated unit with
-clamped inputs. A layer may share another layer's weights; its cache is its own. The configuration gives each layer its own
-sizes.
+Norms are RMS norms with weights around one. The attention has grouped heads with normalised queries and keys, no positions,
+a window beside the first tokens, which stay visible, a sink in the softmax, and a gate on its output; the feed-forward is a
+gated unit with clamped inputs. A layer may share another layer's weights; its cache is its own. The configuration gives each
+layer its own sizes.
 
 Both sublayers read the same h and end in the same sum, so a layer is two products: `[q | k | v | g | gate | up]` on h and
 `[o | down]` on the attention's and the feed-forward's results side by side.
